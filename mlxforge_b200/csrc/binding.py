@@ -8,7 +8,7 @@ if the library cannot be built or loaded, ``kernels()`` raises.
 from __future__ import annotations
 
 import ctypes
-from ctypes import c_float, c_int, c_longlong, c_void_p
+from ctypes import c_double, c_float, c_int, c_longlong, c_void_p
 from typing import Optional
 
 from . import build as _build
@@ -56,7 +56,8 @@ _SIGNATURES = {
     "mf_mid_rows_max": [],
     "mf_mid_rows_linear": [_P, _P, _P, c_int, _P, c_int, c_int, c_int, c_int, _P, _P],
     "mf_embed_positions": [_P, c_int, _P, _P, _P, _P, c_int, c_int, c_int, c_int, _P],
-    "mf_hyper_update_norm": [_P, _P, c_int, _P, _P, _P, _P, _P, c_float, c_int, _P, c_int, _P, c_int, c_int, c_int, _P],
+    "mf_hyper_update_norm": [_P, _P, c_int, _P, _P, _P, _P, _P, c_float, c_int, _P, c_int, _P, c_int, c_int, c_int,
+                             _P, _P, _P, c_float, c_float, c_float, _P],
     "mf_attention_talking": [_P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, c_int,
                              c_float, c_float, _P, c_int, c_int, _P],
     "mf_biased_kv_store": [_P, c_int, _P, _P, _P, _P, c_int, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int,
@@ -72,7 +73,7 @@ _SIGNATURES = {
     "mf_conv_input": [_P, c_int, c_int, _P, c_int, _P, c_longlong, c_longlong, _P, _P, _P, _P, c_int, _P, c_int, _P],
     "mf_postnorm_add": [_P, c_int, c_int, _P, c_float, _P, c_float, c_int, _P, c_float, _P],
     "mf_qk_norm_rope": [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, _P, _P, _P,
-                        _P, _P, _P, _P, _P, _P, _P, c_int, c_int, _P, _P, _P, c_int, _P],
+                        _P, _P, _P, _P, c_int, c_float, c_double, _P, _P, _P, c_int, c_int, _P, _P, _P, c_int, _P],
     "mf_rotate_rows": [_P, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, c_float, _P],
     "mf_moe_route": [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P, _P, _P, _P],
     "mf_moe_rows": [_P, _P, _P, c_int, _P, _P, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_int, _P],
@@ -120,6 +121,17 @@ _SIGNATURES = {
                                 c_int, c_int, _P],
     "mf_retention_output": [_P, c_int, c_longlong, _P, c_int, c_longlong, c_float, _P, c_int, c_int, c_int, _P, c_int,
                             c_int, _P],
+    "mf_conv_act": [_P, c_int, c_int, c_int, _P, _P, c_int, c_int, _P, c_longlong, c_longlong, _P, _P, _P, _P, c_int, _P,
+                    _P, c_int, _P],
+    "mf_decay_parts": [c_int, c_int],
+    "mf_decay_blocks": [c_int, c_int, c_int],
+    "mf_decay_recurrence": [_P, c_int, _P, c_int, _P, c_int, _P, c_int, _P, c_int, _P, _P, _P, c_float, _P, c_longlong, _P,
+                            _P, _P, _P, c_longlong, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
+    "mf_gated_norm": [_P, c_int, c_longlong, _P, c_longlong, _P, c_int, c_float, _P, c_int, c_int, c_int, c_int, c_int, _P],
+    "mf_scan_blocks": [c_int, c_int],
+    "mf_selective_scan": [_P, _P, c_int, _P, _P, c_int, _P, c_int, _P, _P, _P, c_longlong, _P, _P, _P, _P, _P, c_int, c_int,
+                          _P, c_int, c_int, c_int, c_int, _P],
+    "mf_low_rank": [_P, c_int, _P, c_int, _P, c_int, c_float, _P, c_int, c_int, c_int, _P],
 }
 
 MF_ERRORS = {10001: "a size or option this kernel does not take", 10002: "an unsupported dtype"}

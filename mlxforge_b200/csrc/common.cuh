@@ -210,6 +210,14 @@ enum MfKernel {
   MF_K_ROTATE_ROWS,           // heads of a row turned by the position (an attention output turned back)
   MF_K_GDELTA_PREPARE,        // operands of the generalized delta rule: unit keys, removal rates, tanh of the low rank
   MF_K_GDELTA_RECURRENCE,     // its state, token after token
+  MF_K_CONV_ACT,              // short causal convolution with bias and activation on columns of the projections
+  MF_K_DECAY_RECURRENCE,      // a state per head with a decay per head or per key channel and token
+  MF_K_DECAY_LOCAL,           // the same over segments from a zero state
+  MF_K_SCAN_COMBINE,          // the states at the starts of the segments
+  MF_K_GATED_NORM,            // gate, RMS norm in groups and weight of a read-out, gate before or after the norm
+  MF_K_SELECTIVE_SCAN,        // a state per channel with token-dependent decay and input weights
+  MF_K_SCAN_LOCAL,            // the same over segments from a zero state
+  MF_K_LOW_RANK,              // a product with a narrow operand and the decay made of it
   MF_K_COUNT
 };
 extern unsigned long long g_mf_kernel_launches[MF_K_COUNT];

@@ -16,6 +16,8 @@ const char* const kNames[MF_K_COUNT] = {
     "head_linear_mma",  "retention_prepare", "retention_recurrence", "retention_chunked", "retention_output",
     "unary_act",        "gemm_tc_act",      "conv_input",       "postnorm_add",     "qk_norm_rope",
     "rotate_rows",      "gdelta_prepare",   "gdelta_recurrence",
+    "conv_act",         "decay_recurrence", "decay_local",      "scan_combine",     "gated_norm",
+    "selective_scan",   "scan_local",       "low_rank",
 };
 int g_sm_count[MF_MAX_DEVICES] = {};
 }  // namespace

@@ -8,6 +8,9 @@
 // stores the streams, reads them with `in` and normalises.  S = 1 with mix = out = in = 1 is
 // the ordinary residual sum.
 //
+// The result y may come as two branches that are still to be normalised and added (HsPair):
+// y = s1 rms(y1) w1 + s2 rms(y2) w2 over the model width; that too happens here.
+//
 // The norm is an RMS norm in groups: the H channels are cut into G equal consecutive groups,
 // each divided by its own sqrt(mean(x^2) + eps), the whole multiplied by w.  G = 1 is RMSNorm.
 //
@@ -19,6 +22,14 @@
 #define HS_MAX_STREAMS 8
 #define HS_MAX_GROUPS 64
 #define HS_THREADS 256
+
+// The second branch of a result and what both pass before they are added; all null: `delta` alone, as it is.
+struct HsPair {
+  const void* second;
+  const float* w1;       // [H]
+  const float* w2;
+  float s1, s2, eps;
+};
 
 template <typename T>
 __global__ void __launch_bounds__(HS_THREADS)
@@ -71,7 +82,7 @@ hyper_update_norm_kernel(float* __restrict__ streams, const TD* __restrict__ del
                          const float* __restrict__ delta_bias, const float* __restrict__ mix,
                          const float* __restrict__ wout, const float* __restrict__ win,
                          const float* __restrict__ w, float eps, int groups, TO* __restrict__ out,
-                         const int* __restrict__ rows, int H, int S) {
+                         const int* __restrict__ rows, int H, int S, HsPair pair) {
   extern __shared__ float u[];      // [H]
   __shared__ float red[32];
   __shared__ float cm[HS_MAX_STREAMS * HS_MAX_STREAMS], co[HS_MAX_STREAMS], ci[HS_MAX_STREAMS];
@@ -89,12 +100,28 @@ hyper_update_norm_kernel(float* __restrict__ streams, const TD* __restrict__ del
   const long long src = rows ? rows[r] : r;
   float* x = streams + src * S * H;
   const TD* d = delta ? delta + src * H : nullptr;
+  const TD* d2 = pair.second ? (const TD*)pair.second + src * H : nullptr;
+  float i1 = 1.f, i2 = 1.f;
+  if (d2) {
+    float a = 0.f, b = 0.f;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+      const float y1 = to_f32<TD>(d[i]), y2 = to_f32<TD>(d2[i]);
+      a = fmaf(y1, y1, a);
+      b = fmaf(y2, y2, b);
+    }
+    a = block_sum(a, red);
+    b = block_sum(b, red);
+    i1 = pair.s1 / sqrtf(a / (float)H + pair.eps);
+    i2 = pair.s2 / sqrtf(b / (float)H + pair.eps);
+  }
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     float xs[HS_MAX_STREAMS];
 #pragma unroll
     for (int s = 0; s < HS_MAX_STREAMS; s++) xs[s] = (s < S) ? x[(long long)s * H + i] : 0.f;
     if (d) {
-      const float y = to_f32<TD>(d[i]) + (delta_bias ? delta_bias[i] : 0.f);
+      float y = to_f32<TD>(d[i]);
+      if (d2) y = y * i1 * pair.w1[i] + to_f32<TD>(d2[i]) * i2 * pair.w2[i];
+      if (delta_bias) y += delta_bias[i];
       float nx[HS_MAX_STREAMS];
 #pragma unroll
       for (int t = 0; t < HS_MAX_STREAMS; t++) {
@@ -133,15 +160,26 @@ hyper_update_norm_kernel(float* __restrict__ streams, const TD* __restrict__ del
   for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = from_f32<TO>(u[i] * ginv[i / gs] * w[i]);
 }
 
+__device__ __forceinline__ void hs_load4(const float* p, float* y) {
+  const float4 v = *reinterpret_cast<const float4*>(p);
+  y[0] = v.x; y[1] = v.y; y[2] = v.z; y[3] = v.w;
+}
+__device__ __forceinline__ void hs_load4(const __nv_bfloat16* p, float* y) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+  y[0] = a.x; y[1] = a.y; y[2] = b.x; y[3] = b.y;
+}
+
 // The same with the channels in groups of four (H and the group size multiples of 4): 16-byte
 // accesses to the streams, and each thread keeps its values of u in registers between the passes.
-template <typename TD, typename TO, int NV>
+template <typename TD, typename TO, int NV, bool PAIR>
 __global__ void __launch_bounds__(HS_THREADS)
 hyper_update_norm_vec_kernel(float* __restrict__ streams, const TD* __restrict__ delta,
                              const float* __restrict__ delta_bias, const float* __restrict__ mix,
                              const float* __restrict__ wout, const float* __restrict__ win,
                              const float* __restrict__ w, float eps, int groups, TO* __restrict__ out,
-                             const int* __restrict__ rows, int H, int S) {
+                             const int* __restrict__ rows, int H, int S, HsPair pair) {
   __shared__ float red[32];
   __shared__ float cm[HS_MAX_STREAMS * HS_MAX_STREAMS], co[HS_MAX_STREAMS], ci[HS_MAX_STREAMS];
   __shared__ float gsum[HS_MAX_GROUPS];
@@ -159,6 +197,54 @@ hyper_update_norm_vec_kernel(float* __restrict__ streams, const TD* __restrict__
   float* x = streams + src * S * H;
   const TD* d = delta ? delta + src * H : nullptr;
   const int gs = H / groups;
+  float y[NV][4];                // the result that is written back
+  if (d) {
+#pragma unroll
+    for (int j = 0; j < NV; j++) {
+      const int i = (j * HS_THREADS + threadIdx.x) * 4;
+      if (i < H) hs_load4(d + i, y[j]);
+      else y[j][0] = y[j][1] = y[j][2] = y[j][3] = 0.f;
+    }
+    if constexpr (PAIR) {
+      float y2[NV][4], a = 0.f, b = 0.f;
+      const TD* d2 = (const TD*)pair.second + src * H;
+#pragma unroll
+      for (int j = 0; j < NV; j++) {
+        const int i = (j * HS_THREADS + threadIdx.x) * 4;
+        if (i < H) hs_load4(d2 + i, y2[j]);
+        else y2[j][0] = y2[j][1] = y2[j][2] = y2[j][3] = 0.f;
+#pragma unroll
+        for (int e = 0; e < 4; e++) {
+          a = fmaf(y[j][e], y[j][e], a);
+          b = fmaf(y2[j][e], y2[j][e], b);
+        }
+      }
+      a = block_sum(a, red);
+      b = block_sum(b, red);
+      const float i1 = pair.s1 / sqrtf(a / (float)H + pair.eps), i2 = pair.s2 / sqrtf(b / (float)H + pair.eps);
+#pragma unroll
+      for (int j = 0; j < NV; j++) {
+        const int i = (j * HS_THREADS + threadIdx.x) * 4;
+        if (i < H) {
+          const float4 w1 = *reinterpret_cast<const float4*>(pair.w1 + i), w2 = *reinterpret_cast<const float4*>(pair.w2 + i);
+          y[j][0] = y[j][0] * i1 * w1.x + y2[j][0] * i2 * w2.x;
+          y[j][1] = y[j][1] * i1 * w1.y + y2[j][1] * i2 * w2.y;
+          y[j][2] = y[j][2] * i1 * w1.z + y2[j][2] * i2 * w2.z;
+          y[j][3] = y[j][3] * i1 * w1.w + y2[j][3] * i2 * w2.w;
+        }
+      }
+    }
+    if (delta_bias) {
+#pragma unroll
+      for (int j = 0; j < NV; j++) {
+        const int i = (j * HS_THREADS + threadIdx.x) * 4;
+        if (i < H) {
+#pragma unroll
+          for (int e = 0; e < 4; e++) y[j][e] += delta_bias[i + e];
+        }
+      }
+    }
+  }
   float u[NV][4];
 #pragma unroll
   for (int j = 0; j < NV; j++) {
@@ -174,9 +260,6 @@ hyper_update_norm_vec_kernel(float* __restrict__ streams, const TD* __restrict__
         }
       }
       if (d) {
-        float y[4];
-#pragma unroll
-        for (int e = 0; e < 4; e++) y[e] = to_f32<TD>(d[i + e]) + (delta_bias ? delta_bias[i + e] : 0.f);
         float nx[HS_MAX_STREAMS][4];
 #pragma unroll
         for (int t = 0; t < HS_MAX_STREAMS; t++) {
@@ -187,7 +270,7 @@ hyper_update_norm_vec_kernel(float* __restrict__ streams, const TD* __restrict__
 #pragma unroll
               for (int s = 0; s < HS_MAX_STREAMS; s++)
                 if (s < S) a = fmaf(cm[s * S + t], xs[s][e], a);
-              nx[t][e] = fmaf(co[t], y[e], a);
+              nx[t][e] = fmaf(co[t], y[j][e], a);
             }
             if (!rows)
               *reinterpret_cast<float4*>(x + (long long)t * H + i) = make_float4(nx[t][0], nx[t][1], nx[t][2], nx[t][3]);
@@ -237,35 +320,45 @@ hyper_update_norm_vec_kernel(float* __restrict__ streams, const TD* __restrict__
 MF_API int mf_hyper_update_norm(float* streams, const void* delta, int delta_dtype, const float* delta_bias,
                                 const float* mix, const float* wout, const float* win, const float* w, float eps,
                                 int groups, void* out, int out_dtype, const int* rows, int n, int H, int S,
+                                const void* second, const float* w1, const float* w2, float s1, float s2, float pair_eps,
                                 cudaStream_t stream) {
   if (n <= 0) return 0;
   if (S < 1 || S > HS_MAX_STREAMS || groups < 1 || groups > HS_MAX_GROUPS || H % groups) return MF_ERR_BAD_ARG;
+  if (second && (!delta || !w1 || !w2)) return MF_ERR_BAD_ARG;
+  const HsPair pair{second, w1, w2, s1, s2, pair_eps};
   const size_t smem = (size_t)H * sizeof(float);
   if (smem > 200 * 1024) return MF_ERR_BAD_ARG;
   mf_count(MF_K_HYPER_NORM);
+#define HS_VEC(TD, TO, NV, PAIR)                                                                                 \
+  return (int)launch_dep(hyper_update_norm_vec_kernel<TD, TO, NV, PAIR>, dim3(n), dim3(HS_THREADS), 0, stream,   \
+                         streams, (const TD*)delta, delta_bias, mix, wout, win, w, eps, groups, (TO*)out, rows,  \
+                         H, S, pair)
 #define HS_LAUNCH(TD, TO)                                                                                        \
   do {                                                                                                           \
-    const bool vec = H % 4 == 0 && (H / groups) % 4 == 0 && H <= 4 * HS_THREADS * 8 &&                           \
-                     ((uintptr_t)streams & 15) == 0 && ((uintptr_t)w & 15) == 0;                                 \
-    if (vec && H <= 4 * HS_THREADS * 2)                                                                          \
-      return (int)launch_dep(hyper_update_norm_vec_kernel<TD, TO, 2>, dim3(n), dim3(HS_THREADS), 0, stream,      \
-                             streams, (const TD*)delta, delta_bias, mix, wout, win, w, eps, groups, (TO*)out,    \
-                             rows, H, S);                                                                        \
-    if (vec)                                                                                                     \
-      return (int)launch_dep(hyper_update_norm_vec_kernel<TD, TO, 8>, dim3(n), dim3(HS_THREADS), 0, stream,      \
-                             streams, (const TD*)delta, delta_bias, mix, wout, win, w, eps, groups, (TO*)out,    \
-                             rows, H, S);                                                                        \
+    auto al = [](const void* x) { return ((uintptr_t)x & 15) == 0; };                                            \
+    const bool vec = H % 4 == 0 && (H / groups) % 4 == 0 && H <= 4 * HS_THREADS * 8 && al(streams) && al(w) &&   \
+                     al(delta) && al(second) && al(w1) && al(w2);                                                \
+    if (vec && H <= 4 * HS_THREADS * 2) {                                                                        \
+      if (second) HS_VEC(TD, TO, 2, true);                                                                       \
+      HS_VEC(TD, TO, 2, false);                                                                                  \
+    }                                                                                                            \
+    if (vec) {                                                                                                   \
+      if (second) HS_VEC(TD, TO, 8, true);                                                                       \
+      HS_VEC(TD, TO, 8, false);                                                                                  \
+    }                                                                                                            \
     if (smem > 48 * 1024) {                                                                                      \
       cudaError_t e = cudaFuncSetAttribute(hyper_update_norm_kernel<TD, TO>,                                     \
                                            cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);              \
       if (e != cudaSuccess) return (int)e;                                                                       \
     }                                                                                                            \
     return (int)launch_dep(hyper_update_norm_kernel<TD, TO>, dim3(n), dim3(HS_THREADS), smem, stream, streams,   \
-                           (const TD*)delta, delta_bias, mix, wout, win, w, eps, groups, (TO*)out, rows, H, S);  \
+                           (const TD*)delta, delta_bias, mix, wout, win, w, eps, groups, (TO*)out, rows, H, S,   \
+                           pair);                                                                                \
   } while (0)
   if (delta_dtype == MF_F32 && out_dtype == MF_F32) HS_LAUNCH(float, float);
   if (delta_dtype == MF_BF16 && out_dtype == MF_BF16) HS_LAUNCH(__nv_bfloat16, __nv_bfloat16);
   if (delta_dtype == MF_F32 && out_dtype == MF_BF16) HS_LAUNCH(float, __nv_bfloat16);
 #undef HS_LAUNCH
+#undef HS_VEC
   return MF_ERR_BAD_DTYPE;
 }

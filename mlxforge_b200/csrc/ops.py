@@ -651,17 +651,23 @@ def embed_positions(table: torch.Tensor, tokens: torch.Tensor, positions: torch.
 def hyper_update_norm(streams: torch.Tensor, delta: Optional[torch.Tensor], delta_bias: Optional[torch.Tensor],
                       mix: Optional[torch.Tensor], w_out: Optional[torch.Tensor], w_in: Optional[torch.Tensor],
                       weight: torch.Tensor, eps: float, groups: int, out: torch.Tensor, n_streams: int,
-                      rows: Optional[torch.Tensor] = None) -> None:
+                      rows: Optional[torch.Tensor] = None, pair=None) -> None:
     """Write ``delta`` back into the streams (``x_t <- sum_s mix[s, t] x_s + w_out[t] (delta + bias)``), read
     them (``u = sum_s w_in[s] x_s``) and normalise ``u`` in ``groups`` groups.  ``streams`` is [T, S * H]
-    32-bit; with ``rows`` only those rows are produced and the streams stay as they are."""
-    _need_cuda(streams, delta, delta_bias, mix, w_out, w_in, weight, out, rows)
+    32-bit; with ``rows`` only those rows are produced and the streams stay as they are.  ``pair``: what is
+    written back is ``first_scale rms(delta) first_weight + second_scale rms(second) second_weight`` over the
+    model width, with ``pair`` = (second, first_weight, second_weight, first_scale, second_scale, eps)."""
+    second, w1, w2, s1, s2, pair_eps = pair if pair is not None else (None, None, None, 0.0, 0.0, 0.0)
+    _need_cuda(streams, delta, delta_bias, mix, w_out, w_in, weight, out, rows, second, w1, w2)
+    if second is not None and (delta is None or second.dtype != delta.dtype or second.shape != delta.shape):
+        raise KernelError("hyper_update_norm: the two branches must have one dtype and shape")
     H = out.shape[-1]
     n = out.shape[0]
     check(library().mf_hyper_update_norm(streams.data_ptr(), _ptr(delta), dtype_code(delta) if delta is not None else
                                          dtype_code(out), _ptr(delta_bias), _ptr(mix), _ptr(w_out), _ptr(w_in),
                                          weight.data_ptr(), eps, groups, out.data_ptr(), dtype_code(out), _ptr(rows),
-                                         n, H, n_streams, _stream()), "hyper_update_norm")
+                                         n, H, n_streams, _ptr(second), _ptr(w1), _ptr(w2), s1, s2, pair_eps,
+                                         _stream()), "hyper_update_norm")
 
 
 # ---------------------------------------------------------------------------- attention with talking heads
@@ -794,15 +800,18 @@ def postnorm_add(x: torch.Tensor, y1: torch.Tensor, s1: float, y2: Optional[torc
 def qk_norm_rope(proj: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, v_dim: int, rot: int,
                  values_from_keys: bool, eps: float, magnitude: float, bias, q_w, k_w, inv_f, inv_d, vinv_f, vinv_d,
                  batch, block_table: torch.Tensor, page_size: int, q_out: torch.Tensor, k_pool: torch.Tensor,
-                 v_pool: torch.Tensor, write_kv: bool) -> None:
-    """Biases, the norms of queries and keys over their whole projections, the rotation (cosine and sine times
+                 v_pool: torch.Tensor, write_kv: bool, per_head: bool = False, temp_coef: float = 0.0,
+                 temp_every: float = 1.0) -> None:
+    """Biases, the norms of queries and keys over their whole projections (``per_head``: over every head, the
+    weights [head_dim] shared by the heads), the queries times ``1 + temp_coef ln(floor((position + 1) /
+    temp_every) + 1)``, the rotation (cosine and sine times
     ``magnitude``), the values (own, optionally rotated with ``vinv_*``, or the keys as projected) and the cache
     write."""
     _need_cuda(proj, q_out, k_pool, v_pool, bias, q_w, k_w, inv_f, inv_d, vinv_f, vinv_d, block_table)
     check(library().mf_qk_norm_rope(proj.data_ptr(), proj.shape[1], dtype_code(proj), dtype_code(q_out), proj.shape[0], n_heads, n_kv,
                                     head_dim, v_dim, rot, 1 if values_from_keys else 0, eps, magnitude, _ptr(bias),
                                     _ptr(q_w), _ptr(k_w), _ptr(inv_f), _ptr(inv_d), _ptr(vinv_f), _ptr(vinv_d),
-                                    batch.positions.data_ptr(), batch.seq_of_token.data_ptr(), block_table.data_ptr(),
+                                    int(per_head), temp_coef, temp_every, batch.positions.data_ptr(), batch.seq_of_token.data_ptr(), block_table.data_ptr(),
                                     block_table.shape[1], page_size, q_out.data_ptr(), k_pool.data_ptr(),
                                     v_pool.data_ptr(), int(write_kv), _stream()), "qk_norm_rope")
 
@@ -814,6 +823,134 @@ def rotate_rows(x: torch.Tensor, n_heads: int, d: int, rot: int, positions: torc
     _need_cuda(x, positions, inv_f, inv_d)
     check(library().mf_rotate_rows(x.data_ptr(), dtype_code(x), x.shape[0], n_heads, d, rot, positions.data_ptr(),
                                    _ptr(inv_f), _ptr(inv_d), sign, _stream()), "rotate_rows")
+
+
+# ---------------------------------------------------------------------------- state-space and linear recurrences
+
+def conv_act(x: torch.Tensor, ld: int, w: torch.Tensor, bias: Optional[torch.Tensor], silu: bool, state: torch.Tensor,
+             tail_off: int, batch, out: torch.Tensor, out2: Optional[torch.Tensor] = None) -> None:
+    """``out`` [T, C] (32-bit) = act(bias + the causal convolution of ``x``'s first C columns over time): ``x``
+    points at the first column (32-bit rows ``ld`` floats apart), ``w`` [C, taps], the last taps-1 inputs of
+    every sequence in its slot of ``state`` from float ``tail_off`` on; they move on after they were read.
+    ``out2``: the same once more, in its dtype."""
+    _need_cuda(w, bias, state, out, out2)
+    T, C = out.shape
+    taps = w.shape[1]
+    check(library().mf_conv_act(x.data_ptr(), ld, T, C, w.data_ptr(), _ptr(bias), taps, int(silu), state.data_ptr(),
+                                state.stride(0), tail_off, batch.seq_of_token.data_ptr(), batch.seq_q_start.data_ptr(),
+                                batch.seq_q_len.data_ptr(), batch.slots.data_ptr(), batch.n_seqs, out.data_ptr(),
+                                _ptr(out2), dtype_code(out2) if out2 is not None else F32, _stream()), "conv_act",
+          launches=2 if taps > 1 and T != batch.n_seqs else 1)
+
+
+SCAN_TARGET_BLOCKS = 888      # blocks a recurrence over a long portion is cut up for: six for every SM
+
+
+def scan_segments(batch, blocks: int, state_floats: int, min_tokens: int, piece: int = 8):
+    """(number of segments, their length) into which a linear recurrence cuts the step's longest portion:
+    as many as fill the GPU beside the ``blocks`` blocks that a sequence has anyway, none shorter than
+    ``min_tokens``, within 256 MB of states; one segment where every portion is short."""
+    longest = max(batch.q_len)
+    if longest < 2 * min_tokens:
+        return 1, longest
+    n_long = sum(1 for n in batch.q_len if n >= 2 * min_tokens)
+    n = min(-(-SCAN_TARGET_BLOCKS // (blocks * n_long)), longest // min_tokens,
+            max(1, (64 << 20) // (batch.n_seqs * state_floats)))
+    if n < 2:
+        return 1, longest
+    length = -(-longest // n)
+    length = -(-length // piece) * piece
+    return -(-longest // length), length
+
+
+def decay_parts(dim: int, vdim: int) -> int:
+    """How many partial read-outs ``decay_recurrence`` writes for these sizes; ``gated_norm`` sums them."""
+    return int(library().mf_decay_parts(dim, vdim))
+
+
+def decay_blocks(n_heads: int, dim: int, vdim: int) -> int:
+    """Blocks of ``decay_recurrence`` per sequence and segment."""
+    return int(library().mf_decay_blocks(n_heads, dim, vdim))
+
+
+def decay_recurrence(q: torch.Tensor, q_ld: int, k: torch.Tensor, k_ld: int, v: torch.Tensor, v_ld: int,
+                     state: torch.Tensor, batch, o_out: torch.Tensor, n_heads: int, n_qk: int, dim: int, vdim: int,
+                     alpha: Optional[torch.Tensor] = None, dt: Optional[torch.Tensor] = None, dt_ld: int = 0,
+                     dt_bias: Optional[torch.Tensor] = None, a_log: Optional[torch.Tensor] = None,
+                     skip: Optional[torch.Tensor] = None, q_scale: float = 1.0, segments=(1, 0), scratch=None) -> None:
+    """``S <- diag(a) S + k v^T; o = q_scale S^T q (+ skip v)`` per head from the slot's state, with ``a`` =
+    ``alpha`` [T, n_heads * dim], or with the step sizes ``dt`` = softplus(logit + dt_bias) of every head
+    ``a = exp(-exp(a_log) dt)`` and ``v`` times dt.  q, k, v and the logits are the first element of the first
+    token of 32-bit rows ``*_ld`` floats apart; query head h reads q and k of head h // (n_heads // n_qk).
+    ``o_out`` [``decay_parts``, T, n_heads * vdim].  ``segments`` = (number, length) from ``scan_segments``;
+    with more than one, ``scratch`` = (states, decays)."""
+    _need_cuda(state, o_out, alpha, dt_bias, a_log, skip)
+    if o_out.dim() != 3 or o_out.shape[0] != decay_parts(dim, vdim):
+        raise KernelError("decay_recurrence: o_out must hold decay_parts(...) partial read-outs")
+    n_seg, seg_len = segments
+    seg_len = seg_len or max(batch.q_len)
+    s_state = s_decay = None
+    if n_seg > 1:
+        s_state, s_decay = scratch
+        per = n_heads * dim if alpha is not None else n_heads
+        if s_state.numel() < batch.n_seqs * n_seg * n_heads * dim * vdim or s_decay.numel() < batch.n_seqs * n_seg * per:
+            raise KernelError("decay_recurrence: scratch too small")
+    check(library().mf_decay_recurrence(q.data_ptr(), q_ld, k.data_ptr(), k_ld, v.data_ptr(), v_ld, _ptr(alpha),
+                                        alpha.shape[1] if alpha is not None else 0, _ptr(dt), dt_ld, _ptr(dt_bias),
+                                        _ptr(a_log), _ptr(skip), q_scale, state.data_ptr(), state.stride(0),
+                                        batch.seq_q_start.data_ptr(), batch.seq_q_len.data_ptr(), batch.slots.data_ptr(),
+                                        o_out.data_ptr(), o_out.stride(0), _ptr(s_state), _ptr(s_decay), seg_len, n_seg,
+                                        batch.n_seqs, n_heads, n_qk, dim, vdim, _stream()), "decay_recurrence",
+          launches=3 if n_seg > 1 else 1)
+
+
+def gated_norm(x: torch.Tensor, gate: torch.Tensor, gate_ld: int, weight: torch.Tensor, eps: float, out: torch.Tensor,
+               groups: int, gate_first: bool) -> None:
+    """``x`` [parts, T, width] summed over the parts; the row's ``groups`` equal parts divided by their own root
+    mean square, times ``weight`` ([width], or [width / groups] shared by the groups) and silu of ``gate`` (32-bit
+    rows ``gate_ld`` floats apart), which multiplies before the norm (``gate_first``) or after it."""
+    _need_cuda(x, weight, out)
+    check(library().mf_gated_norm(x.data_ptr(), x.shape[0], x.stride(0), gate.data_ptr(), gate_ld, weight.data_ptr(),
+                                  weight.numel(), eps, out.data_ptr(), dtype_code(out), x.shape[1], x.shape[2], groups,
+                                  int(gate_first), _stream()), "gated_norm")
+
+
+def scan_blocks(channels: int, n_state: int) -> int:
+    """Blocks of ``selective_scan`` per sequence and segment (0: more states than it takes)."""
+    return int(library().mf_scan_blocks(channels, n_state))
+
+
+def selective_scan(u: torch.Tensor, dt: torch.Tensor, dt_ld: int, dt_bias: torch.Tensor, z: torch.Tensor, z_ld: int,
+                   bc: torch.Tensor, bc_ld: int, A: torch.Tensor, D: torch.Tensor, state: torch.Tensor, batch,
+                   out: torch.Tensor, n_state: int, segments=(1, 0), scratch=None) -> None:
+    """``S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c u_c B_n; out_c = (sum_n S[c, n] C_n + D_c u_c) silu(z_c)`` from
+    the slot's state, ``dt`` = softplus(logit + dt_bias).  ``bc`` points at B of the first token, C behind it.
+    ``segments`` and ``scratch`` as in ``decay_recurrence`` (states, sums of step sizes)."""
+    _need_cuda(u, dt_bias, A, D, state, out)
+    T, channels = u.shape
+    n_seg, seg_len = segments
+    seg_len = seg_len or max(batch.q_len)
+    s_state = s_dt = None
+    if n_seg > 1:
+        s_state, s_dt = scratch
+        if s_state.numel() < batch.n_seqs * n_seg * channels * n_state or s_dt.numel() < batch.n_seqs * n_seg * channels:
+            raise KernelError("selective_scan: scratch too small")
+    check(library().mf_selective_scan(u.data_ptr(), dt.data_ptr(), dt_ld, dt_bias.data_ptr(), z.data_ptr(), z_ld,
+                                      bc.data_ptr(), bc_ld, A.data_ptr(), D.data_ptr(), state.data_ptr(), state.stride(0),
+                                      batch.seq_q_start.data_ptr(), batch.seq_q_len.data_ptr(), batch.slots.data_ptr(),
+                                      _ptr(s_state), _ptr(s_dt), seg_len, n_seg, out.data_ptr(), dtype_code(out),
+                                      batch.n_seqs, channels, n_state, _stream()), "selective_scan",
+          launches=3 if n_seg > 1 else 1)
+
+
+def low_rank(low: torch.Tensor, ld: int, wt: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor,
+             decay_tau: Optional[float] = None) -> None:
+    """``out`` [T, n] (32-bit) = bias + low wt for ``wt`` [R, n] and 32-bit rows of R numbers ``ld`` floats apart;
+    with ``decay_tau`` sigmoid(.)^(1/decay_tau) of it."""
+    _need_cuda(wt, bias, out)
+    check(library().mf_low_rank(low.data_ptr(), ld, wt.data_ptr(), dtype_code(wt), _ptr(bias),
+                                0 if decay_tau is None else 1, 1.0 if decay_tau is None else decay_tau, out.data_ptr(),
+                                out.shape[0], wt.shape[0], out.shape[1], _stream()), "low_rank")
 
 
 # ---------------------------------------------------------------------------- mixture of experts

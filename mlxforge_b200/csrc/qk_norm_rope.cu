@@ -1,9 +1,11 @@
 // Queries, keys and values on their way from the projection into the attention, for mixers that
-// normalise queries and keys over the WHOLE projection (all heads at once) before the rotation:
+// normalise queries and keys over the WHOLE projection (all heads at once) or PER HEAD before the rotation:
 //
-//   q = rms(Wq h + bq) gq ,  k = rms(Wk h + bk) gk         (one root mean square over all rows of q, one over k)
+//   q = rms(Wq h + bq) gq ,  k = rms(Wk h + bk) gk         (one root mean square over all rows of q, one over k;
+//                                                           per head: one over each head's rows, the weight shared)
 //   rotation of the first `rot` channels of every head, pair (i, i + rot/2), by position * inv[i];
 //   cosine and sine both times `magnitude`
+//   queries optionally times 1 + coef ln(floor((position + 1) / every) + 1)
 //   values: the row's own value heads, optionally rotated over all their vd channels (pair (m, m + vd/2)
 //   by position * vinv[m]), or the keys as projected (with their bias, before norm and rotation)
 //
@@ -21,8 +23,11 @@ struct QkPrepare {
   int v_mode;                 // 0: own values, 1: the keys as projected
   float eps, magnitude;
   const float* bias;          // [nq + nk (+ nv)] or null
-  const float* q_w;           // [nq] or null (no norm)
-  const float* k_w;           // [nk] or null
+  int per_head;               // a norm per head; the weights are then [hd], shared by the heads
+  float temp_coef;            // 0: queries keep their temperature
+  double temp_every;
+  const float* q_w;           // [nq] ([hd] per head) or null (no norm)
+  const float* k_w;           // [nk] ([hd] per head) or null
   const float* inv_f;         // [rot/2]
   const double* inv_d;
   const float* vinv_f;        // [vd/2] or null: values are not rotated
@@ -43,6 +48,15 @@ qk_norm_rope_kernel(const TP* __restrict__ proj, int ld, QkPrepare p, const int*
   const int half = p.rot >> 1, vhalf = p.vinv_f || p.vinv_d ? p.vd >> 1 : 0;
   float* cs = qs + nq + nk + nv;      // [half] cos, [half] sin
   float* vcs = cs + 2 * half;         // [vhalf] cos, [vhalf] sin
+  float* hinv = vcs + 2 * vhalf;      // [n_heads + n_kv] inverse root mean squares per head
+  __shared__ float temp_s;
+  if (threadIdx.x == 0) {
+    temp_s = 1.0f;
+    if (p.temp_coef != 0.f) {
+      const double m = floor(((double)pos + 1.0) / p.temp_every) + 1.0;
+      temp_s = 1.0f + p.temp_coef * (sizeof(T) == 4 ? (float)log(m) : logf((float)m));
+    }
+  }
   for (int j = threadIdx.x; j < half; j += blockDim.x) {
     float c, s;
     rotary_cs(pos, j, p.inv_f, p.inv_d, c, s);
@@ -63,8 +77,19 @@ qk_norm_rope_kernel(const TP* __restrict__ proj, int ld, QkPrepare p, const int*
   sq = block_sum(sq, red);
   sk = block_sum(sk, red);
   __syncthreads();
-  const float iq = p.q_w ? 1.0f / sqrtf(sq / (float)nq + p.eps) : 1.0f;
-  const float ik = p.k_w ? 1.0f / sqrtf(sk / (float)nk + p.eps) : 1.0f;
+  const float temp = temp_s;
+  const float iq = (p.q_w && !p.per_head ? 1.0f / sqrtf(sq / (float)nq + p.eps) : 1.0f) * temp;
+  const float ik = p.k_w && !p.per_head ? 1.0f / sqrtf(sk / (float)nk + p.eps) : 1.0f;
+  if (p.per_head) {
+    const int lane = threadIdx.x & 31;
+    for (int h = threadIdx.x >> 5; h < p.n_heads + p.n_kv; h += blockDim.x >> 5) {
+      float ss = 0.f;
+      for (int d = lane; d < p.hd; d += 32) ss = fmaf(qs[h * p.hd + d], qs[h * p.hd + d], ss);
+      ss = warp_sum(ss);
+      if (lane == 0) hinv[h] = 1.0f / sqrtf(ss / (float)p.hd + p.eps) * (h < p.n_heads ? temp : 1.0f);
+    }
+    __syncthreads();
+  }
   // queries and keys: `half` pairs and hd - rot channels that pass, per head
   const int per_head = p.hd - half;
   const int heads = p.n_heads + (write_kv ? p.n_kv : 0);
@@ -73,8 +98,8 @@ qk_norm_rope_kernel(const TP* __restrict__ proj, int ld, QkPrepare p, const int*
     const bool is_k = h >= p.n_heads;
     const int base = h * p.hd;                  // the keys follow the queries in the row
     const float* w = is_k ? p.k_w : p.q_w;
-    const int wb = is_k ? base - nq : base;
-    const float inv = is_k ? ik : iq;
+    const int wb = p.per_head ? 0 : is_k ? base - nq : base;
+    const float inv = p.per_head ? hinv[h] : is_k ? ik : iq;
     const long long off = is_k ? paged_offset(pk, seq, pos, h - p.n_heads) : 0;
     T* dst = is_k ? k_pool + off : q_out + (long long)t * nq + base;
     if (j < half) {
@@ -112,7 +137,7 @@ qk_norm_rope_kernel(const TP* __restrict__ proj, int ld, QkPrepare p, const int*
 MF_API int mf_qk_norm_rope(const void* proj, int ld, int dtype, int out_dtype, int T, int n_heads, int n_kv, int hd, int vd, int rot,
                            int v_mode, float eps, float magnitude, const float* bias, const float* q_w,
                            const float* k_w, const float* inv_f, const double* inv_d, const float* vinv_f,
-                           const double* vinv_d, const int* positions, const int* seq_of_token,
+                           const double* vinv_d, int per_head, float temp_coef, double temp_every, const int* positions, const int* seq_of_token,
                            const int* block_table, int bt_stride, int page_size, void* q_out, void* k_pool,
                            void* v_pool, int write_kv, cudaStream_t stream) {
   if (T <= 0) return 0;
@@ -120,11 +145,13 @@ MF_API int mf_qk_norm_rope(const void* proj, int ld, int dtype, int out_dtype, i
   if (v_mode < 0 || v_mode > 1 || (v_mode == 1 && vd != hd) || vd <= 0) return MF_ERR_BAD_ARG;
   const bool vrot = vinv_f || vinv_d;
   if (vrot && (vd & 1)) return MF_ERR_BAD_ARG;
-  const QkPrepare p{n_heads, n_kv, hd, vd, rot, v_mode, eps, magnitude, bias, q_w, k_w, inv_f, inv_d, vinv_f, vinv_d};
+  if ((per_head && (!q_w || !k_w)) || (temp_coef != 0.f && !(temp_every > 0.0))) return MF_ERR_BAD_ARG;
+  const QkPrepare p{n_heads, n_kv, hd, vd, rot, v_mode, eps, magnitude, bias, per_head, temp_coef, temp_every, q_w, k_w,
+                    inv_f, inv_d, vinv_f, vinv_d};
   const PagedView pk{block_table, bt_stride, page_size, n_kv, hd};
   const PagedView pvv{block_table, bt_stride, page_size, n_kv, vd};
   const int n = n_heads * hd + n_kv * hd + (v_mode == 0 ? n_kv * vd : 0);
-  const size_t smem = (size_t)(n + rot + (vrot ? vd : 0) + 4) * sizeof(float);
+  const size_t smem = (size_t)(n + rot + (vrot ? vd : 0) + n_heads + n_kv + 4) * sizeof(float);
   if (smem > 200 * 1024) return MF_ERR_BAD_ARG;
   mf_count(MF_K_QK_NORM_ROPE);
 #define QK_LAUNCH(TP, TT)                                                                                          \

@@ -3,5 +3,5 @@ from .base import (BLOCKS, CONNECTIONS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS
                    FixedState, LayerSpec, Mixer, ModelSpec, Norm, PagedKV, Part, PartSpec, PositionEncoding,
                    ScaledPair, ScheduleItem, TensorSpec, build_part, register_block, register_connection, register_embedding,
                    register_feed_forward, register_head, register_mixer, register_norm, register_position)
-from . import (attention, block, connections, delta_rule, embedding, latent_attention, mlp, moe, norms,  # noqa: F401
-               retention, rope, side_by_side, talking_attention)                                                  # (register the built-in parts)
+from . import (attention, block, connections, delta_rule, embedding, gated_linear, latent_attention, mlp, moe,  # noqa: F401
+               norms, retention, rope, side_by_side, state_space, talking_attention)                           # (register the built-in parts)

@@ -251,11 +251,14 @@ _NORMED_NAMES = {"q": "q", "k": "k", "v": "v", "o": "o", "q_bias": "q.b", "k_bia
 @register_mixer("normed_attention")
 class NormedAttention(Mixer):
     """Grouped-query attention whose queries and keys are normalised over their WHOLE projections (one root
-    mean square over all heads' rows of q, one over k's, each with a plain weight of that size) before they
-    are rotated.  Every option is a parameter:
+    mean square over all heads' rows of q, one over k's, each with a plain weight of that size) or per head
+    before they are rotated.  Every option is a parameter:
 
     * ``bias``: q and k projections have biases (added in 32-bit before the norm);
-    * ``qk_norm``: ``"whole"`` or None;
+    * ``qk_norm``: ``"whole"``, ``"head"`` (a root mean square per head, weights of size ``head_dim`` shared by the
+      heads) or None;
+    * ``query_temperature``: ``{"coef", "every"}`` - the query at position p is multiplied by
+      ``1 + coef ln(floor((p + 1) / every) + 1)``;
     * ``rotary``: ``{"dims", "base", "scaling"}`` - half-split pairs over the first ``dims`` channels of a head;
       ``scaling`` None, ``{"factor"}`` (every frequency divided by it) or ``{"factor", "original", "fast",
       "slow"}`` (the stretched table, cosine and sine times ``0.1 ln(factor) + 1``);
@@ -289,8 +292,12 @@ class NormedAttention(Mixer):
         self.names = dict(_NORMED_NAMES, **(p.get("names") or {}))
         if self.values not in ("own", "keys"):
             raise ValueError(f"normed_attention: values must be 'own' or 'keys', got '{self.values}'")
-        if self.qk_norm not in (None, "whole"):
-            raise ValueError(f"normed_attention: qk_norm must be 'whole' or None, got '{self.qk_norm}'")
+        if self.qk_norm not in (None, "whole", "head"):
+            raise ValueError(f"normed_attention: qk_norm must be 'whole', 'head' or None, got '{self.qk_norm}'")
+        temp = p.get("query_temperature") or {}
+        self.temp_coef, self.temp_every = float(temp.get("coef", 0.0)), float(temp.get("every", 1.0))
+        if not self.temp_every > 0:
+            raise ValueError(f"normed_attention: query_temperature.every must be positive, got {self.temp_every}")
         if self.n_kv <= 0 or self.n_heads % self.n_kv:
             raise ValueError("n_heads must be a multiple of n_kv_heads")
         if self.values == "keys" and self.vd != self.hd:
@@ -333,8 +340,9 @@ class NormedAttention(Mixer):
             specs[self._n("q_bias")] = TensorSpec((nq,), role="vector")
             specs[self._n("k_bias")] = TensorSpec((nk,), role="vector")
         if self.qk_norm:
-            specs[self._n("q_norm")] = TensorSpec((nq,), role="vector")
-            specs[self._n("k_norm")] = TensorSpec((nk,), role="vector")
+            head = self.qk_norm == "head"
+            specs[self._n("q_norm")] = TensorSpec((self.hd if head else nq,), role="vector")
+            specs[self._n("k_norm")] = TensorSpec((self.hd if head else nk,), role="vector")
         return specs
 
     def bind(self, tensors) -> None:
@@ -364,9 +372,13 @@ class NormedAttention(Mixer):
         table = batch.block_table(cache.group)
         ops.qk_norm_rope(proj, self.n_heads, self.n_kv, self.hd, self.vd, self.rot, self.values == "keys", self.eps,
                          self.magnitude, self.b_in, self.q_w, self.k_w, self.inv_f, self.inv_d, self.vinv_f, self.vinv_d,
-                         batch, table, cache.page_size, q, cache.k, cache.v, writes_cache)
+                         batch, table, cache.page_size, q, cache.k, cache.v, writes_cache, self.qk_norm == "head",
+                         self.temp_coef, self.temp_every)
         o = rt.buffer("nattn.o", (T, self.n_heads * self.vd))
-        softcap_attention(rt, batch, q, cache, o, self.n_heads, self.scale, self.window, self.softcap)
+        if not (self.window or self.softcap) and self.vd == self.hd and self.hd % 16 == 0 and self.hd <= 256:
+            paged_attention(rt, batch, q, cache, o, self.n_heads, self.scale, 0)       # nothing beyond the plain kernels
+        else:
+            softcap_attention(rt, batch, q, cache, o, self.n_heads, self.scale, self.window, self.softcap)
         if self.rotate_values:
             ops.rotate_rows(o, self.n_heads, self.vd, self.vd, batch.positions, self.vinv_f, self.vinv_d, -1.0)
         return rt.linear(o, self.w_o, rt.buffer("nattn.delta", (T, self.hidden), torch.float32 if self.out_f32 else None))

@@ -187,6 +187,22 @@ class ScaledPair:
     second_scale: float
 
 
+@dataclass(frozen=True)
+class NormedPair:
+    """The outputs of two branches that ran side by side, each still to be RMS-normalised over the model width
+    (``eps``, plain weights) before their weighted sum is formed:
+    ``first_scale rms(first) first_weight + second_scale rms(second) second_weight``.  The stream write that
+    takes it (``group_rmsnorm``) does all of it in 32-bit in the kernel it runs anyway."""
+
+    first: Any
+    first_weight: Any
+    first_scale: float
+    second: Any
+    second_weight: Any
+    second_scale: float
+    eps: float
+
+
 # --------------------------------------------------------------------------- interfaces
 
 class Part:

@@ -16,7 +16,7 @@ from typing import Dict
 import torch
 
 from ..csrc import ops
-from .base import DeltaPair, Norm, ScaledPair, TensorSpec, register_norm
+from .base import DeltaPair, Norm, NormedPair, ScaledPair, TensorSpec, register_norm
 
 
 @register_norm("rmsnorm")
@@ -88,7 +88,7 @@ class GroupRMSNorm(Norm):
     is RMSNorm).  It also knows models with several residual streams (``streams``): the stream tensor
     is then [T, streams * size], a pending ``StreamWrite`` (see ``connections.py``) is written back
     into the streams first, and the streams are read with the weights ``read`` (None: their plain sum)
-    before the norm; all of it is one kernel."""
+    before the norm; all of it is one kernel.  ``one_plus``: the weight is stored around zero."""
 
     graph_safe = True
 
@@ -99,6 +99,7 @@ class GroupRMSNorm(Norm):
         self.groups = int(params.get("groups", 1) or 1)
         self.streams = int(params.get("streams", 1) or 1)
         self.name = self.prefix + str(params.get("tensor", "weight"))
+        self.one_plus = bool(params.get("one_plus", False))
         if self.groups < 1 or self.size % self.groups:
             raise ValueError(f"group_rmsnorm: {self.size} channels do not divide into {self.groups} groups")
         self.weight = None
@@ -107,7 +108,8 @@ class GroupRMSNorm(Norm):
         return {self.name: TensorSpec((self.size,), role="vector")}
 
     def bind(self, tensors) -> None:
-        self.weight = tensors[self.name].to(torch.float32).contiguous()
+        w = tensors[self.name].to(torch.float32)
+        self.weight = (w + 1.0 if self.one_plus else w).contiguous()
 
     def weight_bytes(self) -> int:
         return self.size * 4
@@ -121,6 +123,9 @@ class GroupRMSNorm(Norm):
         if out is None:
             out = self.rt.buffer("norm.out", (n, self.size))
         w = delta if isinstance(delta, StreamWrite) else StreamWrite(delta)
-        ops.hyper_update_norm(residual, w.delta, w.bias, w.mix, w.out, read, self.weight, self.eps, self.groups, out,
-                              self.streams, rows)
+        d, pair = w.delta, None
+        if isinstance(d, NormedPair):
+            d, pair = d.first, (d.second, d.first_weight, d.second_weight, d.first_scale, d.second_scale, d.eps)
+        ops.hyper_update_norm(residual, d, w.bias, w.mix, w.out, read, self.weight, self.eps, self.groups, out,
+                              self.streams, rows, pair)
         return out

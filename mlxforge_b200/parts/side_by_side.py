@@ -6,6 +6,10 @@ entry) and the pair hands each branch its own lanes.  The two outputs are not ad
 on as a ``ScaledPair`` so that whoever takes them (the norm on the sublayer's output) forms the weighted
 sum in 32-bit in the kernel it runs anyway.
 
+``out_norm`` (``{"eps", "left", "right"}``) puts an RMS norm over the model width with a plain weight (the tensors
+``left`` and ``right`` behind the pair's prefix) on each branch's output before the sum; the pair then travels as a
+``NormedPair``, and the stream write that takes it normalises too.
+
 The branches depend on nothing of each other.  With many tokens in a step (``overlap_min_tokens``, 256 by
 default; 0 switches it off) the right branch is launched on a second stream, forked from and joined back to
 the step's stream by events, so that a branch whose kernels fill a fraction of the GPU (a recurrence that is
@@ -18,7 +22,7 @@ from typing import Dict
 
 import torch
 
-from .base import MIXERS, Mixer, ScaledPair, TensorSpec, build_part, count_needs, flatten_needs, register_mixer
+from .base import MIXERS, Mixer, NormedPair, ScaledPair, TensorSpec, build_part, count_needs, flatten_needs, register_mixer
 
 
 @register_mixer("side_by_side")
@@ -29,6 +33,12 @@ class SideBySide(Mixer):
         self.right = build_part(MIXERS, params["right"], runtime)
         self.left_scale = float(params.get("left_scale", 1.0))
         self.right_scale = float(params.get("right_scale", 1.0))
+        norm = params.get("out_norm")
+        self.out_norm = None
+        if norm:
+            self.hidden = int(params["hidden_size"])
+            self.out_norm = (prefix + str(norm["left"]), prefix + str(norm["right"]), float(norm["eps"]))
+        self.w_left = self.w_right = None
         self.n_left = count_needs(self.left.cache_need())
         self.n_right = count_needs(self.right.cache_need())
         self.overlap_min_tokens = int(params.get("overlap_min_tokens", 256))
@@ -41,11 +51,15 @@ class SideBySide(Mixer):
     def tensor_specs(self) -> Dict[str, TensorSpec]:
         specs = dict(self.left.tensor_specs())
         specs.update(self.right.tensor_specs())
+        if self.out_norm:
+            specs.update({n: TensorSpec((self.hidden,), role="vector") for n in self.out_norm[:2]})
         return specs
 
     def bind(self, tensors) -> None:
         self.left.bind(tensors)
         self.right.bind(tensors)
+        if self.out_norm:
+            self.w_left, self.w_right = (tensors[n].to(torch.float32).contiguous() for n in self.out_norm[:2])
 
     def weight_bytes(self) -> int:
         return self.left.weight_bytes() + self.right.weight_bytes()
@@ -58,6 +72,11 @@ class SideBySide(Mixer):
     def _lanes(lanes, first: int, n: int):
         return None if n == 0 else (lanes[first] if n == 1 else tuple(lanes[first:first + n]))
 
+    def _pair(self, y1, y2):
+        if self.out_norm:
+            return NormedPair(y1, self.w_left, self.left_scale, y2, self.w_right, self.right_scale, self.out_norm[2])
+        return ScaledPair(y1, self.left_scale, y2, self.right_scale)
+
     def forward(self, x, batch, cache, writes_cache: bool = True):
         lanes = cache if isinstance(cache, tuple) else (() if cache is None else (cache,))
         left_lanes, right_lanes = self._lanes(lanes, 0, self.n_left), self._lanes(lanes, self.n_left, self.n_right)
@@ -66,7 +85,7 @@ class SideBySide(Mixer):
         if shared_scratch or not (self.overlap_min_tokens and x.shape[0] >= self.overlap_min_tokens and x.is_cuda):
             y1 = self.left.forward(x, batch, left_lanes, writes_cache)
             y2 = self.right.forward(x, batch, right_lanes, writes_cache)
-            return ScaledPair(y1, self.left_scale, y2, self.right_scale)
+            return self._pair(y1, y2)
         if self._side is None:
             self._side, self._fork, self._join = torch.cuda.Stream(), torch.cuda.Event(), torch.cuda.Event()
         main = torch.cuda.current_stream()
@@ -77,4 +96,4 @@ class SideBySide(Mixer):
             self._join.record(self._side)
         y1 = self.left.forward(x, batch, left_lanes, writes_cache)
         main.wait_event(self._join)                   # whoever takes the pair reads both
-        return ScaledPair(y1, self.left_scale, y2, self.right_scale)
+        return self._pair(y1, y2)
