@@ -423,7 +423,9 @@ class KernelTimes:
                 torch.cuda.synchronize()
                 if i >= 2:
                     ts.append(e0.elapsed_time(e1) * 1e3)
-            out.setdefault(n, []).append((statistics.median(ts), a, k))
+            # the two forms of one recurrence are kinds of their own
+            kind = n if n != "decay_recurrence" else n + (".channel" if k.get("alpha") is not None else ".head")
+            out.setdefault(kind, []).append((statistics.median(ts), a, k))
         return out
 
 
@@ -527,6 +529,23 @@ def kernel_work(name, a, k, info):
                 9.0 * T * nh * dim * dim)
     if name in ("qk_norm_rope", "rotate_rows", "gdelta_prepare", "delta_gates_ex"):
         return (_nbytes(*[t for t in a if hasattr(t, "numel") and t.dim() >= 2 and t.numel() < (1 << 28)]), 0, 0)
+    if name in ("decay_recurrence.head", "decay_recurrence.channel"):
+        state, o, nh, n_qk, dim, vdim = a[6], a[8], a[9], a[10], a[11], a[12]
+        per_token = 2 * n_qk * dim + 2 * nh * vdim + (nh * dim if k.get("alpha") is not None else nh)
+        return (T * per_token * 4 + 2 * info["seqs"] * nh * dim * vdim * 4, 0, 5.0 * T * nh * dim * vdim)
+    if name == "selective_scan":
+        u, out, n_state = a[0], a[12], a[13]
+        # an exponential per state takes the time of 16 FLOPs: 16 a clock and SM, where the FMA lanes do 256
+        return (3 * _nbytes(u) + _nbytes(out) + 2 * info["seqs"] * u.shape[1] * n_state * 4, 0, 16.0 * T * u.shape[1] * n_state)
+    if name == "conv_act":
+        out, out2 = a[8], (a[9] if len(a) > 9 else None)
+        return (2 * _nbytes(out) + _nbytes(out2), 0, 0)
+    if name == "gated_norm":
+        x, out = a[0], a[5]
+        return (_nbytes(x) + out.numel() * 4 + _nbytes(out), 0, 0)
+    if name == "low_rank":
+        wt, out = a[2], a[4]
+        return (_nbytes(wt, out) + T * wt.shape[0] * 4, 0, 2.0 * T * wt.shape[0] * wt.shape[1])
     return (0, 0, 0)
 
 
@@ -868,21 +887,22 @@ def ledinex_notirax_like(z):
             "layers": [dict(attn if i % 2 == 0 else delta, mlp=mlp) for i in range(z["layers"])]}
 
 
-def run_ledinex(args) -> int:
+def run_beside(args, workload, sizes, arms) -> int:
+    """A design beside its neighbour: prefill, decode and the kernels of both at every size.  ``arms(size)`` yields
+    (name, config.json, kernels, chunk of the attention mask)."""
     import torch
     import mlxforge_b200 as mf
     from mlxforge_b200.config import config_from_json
     from mlxforge_b200.csrc import ops
     pk = peaks()
-    out = {"workload": "ledinex", "dtype": "bf16", "peaks": pk,
+    out = {"workload": workload, "dtype": "bf16", "peaks": pk,
            "data": "synthetic: seeded random weights, seeded uniform token ids, random cache contents",
            "fp32_tflops_nominal": round(FP32_TFLOPS_NOMINAL, 1), "sizes": {}}
     sampled = []
-    for key in ([args.size] if args.size else sorted(LEDINEX_SIZES)):
-        z = LEDINEX_SIZES[key]
+    for key in ([args.size] if args.size else sorted(sizes)):
+        z = sizes[key]
         res = {"size": z}
-        for which, cfg_json, names, chunk in (("ledinex", ledinex_config(z), LEDINEX_KERNELS, 0),
-                                              ("notirax_equal_size", ledinex_notirax_like(z), NOTIRAX_KERNELS, z["window"])):
+        for which, cfg_json, names, chunk in arms(z):
             tmp = tempfile.mkdtemp(prefix="mlxforge_bench_")
             try:
                 d = mf.write_random_model(os.path.join(tmp, "model"), config_from_json(cfg_json), seed=0, dtype="bfloat16")
@@ -917,6 +937,63 @@ def run_ledinex(args) -> int:
                      "reasons": sorted({x for c in seen for x in c["reasons"]})}
     print(json.dumps(out))
     return 0
+
+
+def run_ledinex(args) -> int:
+    return run_beside(args, "ledinex", LEDINEX_SIZES,
+                      lambda z: (("ledinex", ledinex_config(z), LEDINEX_KERNELS, 0),
+                                 ("notirax_equal_size", ledinex_notirax_like(z), NOTIRAX_KERNELS, z["window"])))
+
+
+# ---------------------------------------------------------------------------- --workload takavik
+# The Takavik design at sizes that resemble a real model's layers, beside the closest existing model at equal size:
+# a Notirax decoder (several residual streams, attention, a recurrence with short convolutions) with the same
+# width, layers, vocabulary, streams, attention heads and head size, and experts of which a token uses as much
+# feed-forward as Takavik's dense one.  Takavik's layers are mamba2, gla, parallel, mamba2.
+TAKAVIK_SIZES = {
+    "s": dict(width=1024, layers=4, vocab=32768, streams=4, heads=8, kv=2, dim=128, every=1024, inner=2048, state=16,
+              dt_rank=64, conv=4, m_heads=32, m_vdim=64, m_state=128, g_heads=4, g_dim=128, g_vdim=256, g_rank=16, ff=3072,
+              context=4096),
+    "m": dict(width=2048, layers=4, vocab=32768, streams=4, heads=16, kv=4, dim=128, every=1024, inner=4096, state=16,
+              dt_rank=128, conv=4, m_heads=64, m_vdim=64, m_state=128, g_heads=8, g_dim=128, g_vdim=256, g_rank=16, ff=6144,
+              context=4096),
+}
+TAKAVIK_KERNELS = ("embed_positions", "hyper_update_norm", "conv_act", "decay_recurrence", "gated_norm", "low_rank",
+                   "selective_scan", "qk_norm_rope", "attention_prefill", "attention_decode", "attention_prefill_ex",
+                   "attention_decode_ex", "swiglu", "stream_linear", "gemm_bf16")
+
+
+def takavik_config(z):
+    mamba2 = {"type": "mamba2", "mixer": {"heads": z["m_heads"], "vdim": z["m_vdim"], "state": z["m_state"], "groups": 1,
+                                          "norm_groups": 1, "conv": z["conv"]}}
+    gla = {"type": "gla", "mixer": {"heads": z["g_heads"], "dim": z["g_dim"], "vdim": z["g_vdim"], "tau": 16.0,
+                                    "decay_rank": z["g_rank"]}}
+    par = {"type": "parallel", "mixer": {
+        "left": {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+                 "q_temp": {"coef": 0.1, "every": z["every"]}},
+        "right": {"inner": z["inner"], "state": z["state"], "dt_rank": z["dt_rank"], "conv": z["conv"]}}}
+    order = [mamba2, gla, par, mamba2]
+    return {"architecture": "Takavik", "vocab": z["vocab"], "width": z["width"], "streams": z["streams"],
+            "norm": {"eps": 1e-5},
+            "layers": [dict(order[i % 4], mlp={"kind": "dense", "ff": z["ff"]}) for i in range(z["layers"])]}
+
+
+def takavik_notirax_like(z):
+    attn = {"type": "attention", "mixer": {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"],
+                                           "scale": z["dim"] ** -0.5, "mask": {"size": z["context"]}}}
+    delta = {"type": "channel_delta", "mixer": {"heads": z["heads"], "kv_heads": z["heads"], "dim": z["dim"],
+                                                "vdim": z["dim"], "conv": z["conv"], "decay_rank": z["dt_rank"],
+                                                "gate_rank": z["dt_rank"]}}
+    mlp = {"kind": "moe", "expert": {"ff": z["ff"] // 2, "limit": 7.0}, "router": {"experts": 8, "top": 2, "scale": 1.0}}
+    order = [delta, delta, attn, delta]
+    return {"architecture": "Notirax", "vocab": z["vocab"], "width": z["width"], "streams": z["streams"],
+            "norm": {"eps": 1e-5, "groups": 1}, "layers": [dict(order[i % 4], mlp=mlp) for i in range(z["layers"])]}
+
+
+def run_takavik(args) -> int:
+    return run_beside(args, "takavik", TAKAVIK_SIZES,
+                      lambda z: (("takavik", takavik_config(z), TAKAVIK_KERNELS, 0),
+                                 ("notirax_equal_size", takavik_notirax_like(z), NOTIRAX_KERNELS, z["context"])))
 
 
 # Kinds of launches that `--without` leaves out of a decode step, to see what each costs inside it.
@@ -973,13 +1050,13 @@ def main() -> int:
     ap.add_argument("--without", default=None, choices=sorted(LEFT_OUT),
                     help="with --only decode: time the step with the launches of one kind left out (its results are "
                          "wrong; the difference to the full step is what that kind costs inside the step)")
-    ap.add_argument("--workload", default="headline", choices=["headline", "serving", "longctx", "notirax", "luzinex", "rabapel", "ledinex"],
+    ap.add_argument("--workload", default="headline", choices=["headline", "serving", "longctx", "notirax", "luzinex", "rabapel", "ledinex", "takavik"],
                     help="serving: 64 requests on the 3B shape; longctx: 8 x 16,384 tokens on the 8B shape; notirax / "
                          "luzinex: prefill and decode of that design beside the Llama decoder at equal size, per kernel; "
                          "rabapel: the same beside a Luzinex decoder of latent-attention layers at equal size; "
-                         "ledinex: the same beside a Notirax decoder at equal size")
+                         "ledinex / takavik: the same beside a Notirax decoder at equal size")
     ap.add_argument("--size", default=None, choices=sorted(set(NOTIRAX_SIZES) | set(LUZINEX_SIZES) | set(RABAPEL_SIZES)),
-                    help="with --workload notirax, luzinex, rabapel or ledinex: one size only")
+                    help="with --workload notirax, luzinex, rabapel, ledinex or takavik: one size only")
     args = ap.parse_args()
     args.shape_given = args.shape is not None
     args.shape = args.shape or "1b"
@@ -999,6 +1076,8 @@ def main() -> int:
         return run_rabapel(args)
     if args.workload == "ledinex":
         return run_ledinex(args)
+    if args.workload == "takavik":
+        return run_takavik(args)
     if args.workload != "headline":
         return run_workload(args)
 

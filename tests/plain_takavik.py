@@ -213,7 +213,7 @@ def mixer_forward(h, layer, W, eps):
 
 
 def silu_feed_forward(h, W):
-    return lin(silu(lin(h, W["gate"])) * lin(h, W["up"]), W["down"])
+    return _r(lin(silu(_r(lin(h, W["gate"]))) * _r(lin(h, W["up"])), W["down"]))
 
 
 def forward(config, tensors, tokens, layers_out=None):
