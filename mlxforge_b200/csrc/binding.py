@@ -125,6 +125,8 @@ _SIGNATURES = {
                     _P, c_int, _P],
     "mf_decay_parts": [c_int, c_int],
     "mf_decay_blocks": [c_int, c_int, c_int],
+    "mf_decay_resident": [c_int, c_int, c_int, c_int],
+    "mf_scan_resident": [c_int, c_int],
     "mf_decay_recurrence": [_P, c_int, _P, c_int, _P, c_int, _P, c_int, _P, c_int, _P, _P, _P, c_float, _P, c_longlong, _P,
                             _P, _P, _P, c_longlong, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P],
     "mf_gated_norm": [_P, c_int, c_longlong, _P, c_longlong, _P, c_int, c_float, _P, c_int, c_int, c_int, c_int, c_int, _P],

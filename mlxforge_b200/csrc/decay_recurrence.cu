@@ -42,6 +42,8 @@ __device__ __forceinline__ void dc_cp4(void* smem, const void* gmem) {
   const uint32_t a = (uint32_t)__cvta_generic_to_shared(smem);
   asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(a), "l"(gmem) : "memory");
 }
+struct DcTrue { static constexpr bool value = true; };
+struct DcFalse { static constexpr bool value = false; };
 __device__ __forceinline__ float dc_softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 }  // namespace
 
@@ -103,23 +105,30 @@ decay_recurrence_kernel(DecayRec p) {
   const long long s_at = ((long long)h * p.dim + r0) * p.vdim + c0 + cg * DC_TC;
   float* slot_state = p.state + (long long)p.slots[seq] * p.state_stride + s_at;
   const float* S0 = own_segs > 1 ? p.seg_state + ((long long)seq * p.n_seg + seg) * SS + s_at : slot_state;
-  // row i of a thread: ((i / 4) * RL + rl) * 4 + i % 4, so that the lanes of a column read 16-byte pieces side by side
-  float s[DC_TR][DC_TC];
+  // row i of a thread: ((i / 4) * RL + rl) * 4 + i % 4, so that the lanes of a column read 16-byte pieces side by side;
+  // rows 2 i and 2 i + 1 stand in one register pair and are worked on by one instruction
+  f32x2 s[DC_TR / 2][DC_TC];
 #pragma unroll
-  for (int i = 0; i < DC_TR; i++) {
-    const int r = ((i >> 2) * RL + rl) * 4 + (i & 3);
+  for (int i = 0; i < DC_TR / 2; i++) {
+    float x[2][DC_TC];
 #pragma unroll
-    for (int c = 0; c < DC_TC; c++) s[i][c] = 0.f;
-    if (!LOCAL && r < rows_here) {
-      if (p.vec && cg * DC_TC < cols_here) {
-        const float4 x = *reinterpret_cast<const float4*>(S0 + (long long)r * p.vdim);
-        s[i][0] = x.x; s[i][1] = x.y; s[i][2] = x.z; s[i][3] = x.w;
-      } else {
+    for (int e = 0; e < 2; e++) {
+      const int r = ((i >> 1) * RL + rl) * 4 + (i & 1) * 2 + e;
 #pragma unroll
-        for (int c = 0; c < DC_TC; c++)
-          if (cg * DC_TC + c < cols_here) s[i][c] = S0[(long long)r * p.vdim + c];
+      for (int c = 0; c < DC_TC; c++) x[e][c] = 0.f;
+      if (!LOCAL && r < rows_here) {
+        if (p.vec && cg * DC_TC < cols_here) {
+          const float4 f = *reinterpret_cast<const float4*>(S0 + (long long)r * p.vdim);
+          x[e][0] = f.x; x[e][1] = f.y; x[e][2] = f.z; x[e][3] = f.w;
+        } else {
+#pragma unroll
+          for (int c = 0; c < DC_TC; c++)
+            if (cg * DC_TC + c < cols_here) x[e][c] = S0[(long long)r * p.vdim + c];
+        }
       }
     }
+#pragma unroll
+    for (int c = 0; c < DC_TC; c++) s[i][c] = pack2(x[0][c], x[1][c]);
   }
   const int n_chunks = (n + DC_CHUNK - 1) / DC_CHUNK;
   float neg_a = 0.f, dtb = 0.f, skip = 0.f, x_next = 0.f;
@@ -187,9 +196,9 @@ decay_recurrence_kernel(DecayRec p) {
   };
 #pragma unroll
   for (int c = 0; c < DC_STAGES - 1; c++) issue(c);
-  float prod[CHANNEL ? DC_TR : 1];                 // LOCAL: the product of the decays
+  f32x2 prod[CHANNEL ? DC_TR / 2 : 1];             // LOCAL: the product of the decays
 #pragma unroll
-  for (int i = 0; i < (CHANNEL ? DC_TR : 1); i++) prod[i] = 1.f;
+  for (int i = 0; i < (CHANNEL ? DC_TR / 2 : 1); i++) prod[i] = pack2(1.f, 1.f);
   float* o = p.o + (LOCAL ? 0 : (long long)rg * p.part_stride + (long long)h * p.vdim + c0 + cg * DC_TC);
   for (int chunk = 0; chunk < n_chunks; chunk++) {
     asm volatile("cp.async.wait_group %0;\n" ::"n"(DC_STAGES - 2) : "memory");
@@ -197,53 +206,63 @@ decay_recurrence_kernel(DecayRec p) {
     issue(chunk + DC_STAGES - 1);
     const float* st = dc_sm + (size_t)(chunk % DC_STAGES) * DC_CHUNK * TOK;
     const int nt = min(DC_CHUNK, n - chunk * DC_CHUNK);
-    for (int tt = 0; tt < nt; tt += DC_NT) {
+    // four tokens; `whole`: all four are there (the compiler may then overlap them)
+    auto four = [&](int tt, auto whole) {
       float acc[DC_NT * DC_TC];
 #pragma unroll
       for (int i = 0; i < DC_NT * DC_TC; i++) acc[i] = 0.f;
 #pragma unroll
       for (int u = 0; u < DC_NT; u++) {
-        if (tt + u < nt) {
+        if (decltype(whole)::value || tt + u < nt) {
           const float* row = st + (tt + u) * TOK;
           const float4 v4 = *reinterpret_cast<const float4*>(row + V_AT + cg * DC_TC);
           float v[DC_TC] = {v4.x, v4.y, v4.z, v4.w};
-          float ah = 0.f;
+          f32x2 a2 = 0;
           if (!CHANNEL) {
             const float2 ad = *reinterpret_cast<const float2*>(row + S_AT);
-            ah = ad.x;
+            a2 = pack2(ad.x, ad.x);
             if (!LOCAL) {
 #pragma unroll
               for (int c = 0; c < DC_TC; c++) acc[u * DC_TC + c] = skip * v[c];
             }
 #pragma unroll
             for (int c = 0; c < DC_TC; c++) v[c] *= ad.y;
-            if (LOCAL) prod[0] *= ah;
+            if (LOCAL) prod[0] = mul2(prod[0], a2);
+          }
+          f32x2 v2[DC_TC], o2[DC_TC];
+#pragma unroll
+          for (int c = 0; c < DC_TC; c++) {
+            v2[c] = pack2(v[c], v[c]);
+            o2[c] = 0;
           }
 #pragma unroll
           for (int i4 = 0; i4 < DC_TR / 4; i4++) {
-            const float4 k4 = *reinterpret_cast<const float4*>(row + (i4 * RL + rl) * 4);
-            const float kk[4] = {k4.x, k4.y, k4.z, k4.w};
-            float aa[4], qq[4];
+            const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(row + (i4 * RL + rl) * 4);
+            ulonglong2 a4 = make_ulonglong2(a2, a2), q4 = make_ulonglong2(0, 0);
             if (CHANNEL) {
-              const float4 a4 = *reinterpret_cast<const float4*>(row + A_AT + (i4 * RL + rl) * 4);
-              aa[0] = a4.x; aa[1] = a4.y; aa[2] = a4.z; aa[3] = a4.w;
+              a4 = *reinterpret_cast<const ulonglong2*>(row + A_AT + (i4 * RL + rl) * 4);
               if (LOCAL) {
-#pragma unroll
-                for (int e = 0; e < 4; e++) prod[CHANNEL ? i4 * 4 + e : 0] *= aa[e];
+                prod[CHANNEL ? 2 * i4 : 0] = mul2(prod[CHANNEL ? 2 * i4 : 0], a4.x);
+                prod[CHANNEL ? 2 * i4 + 1 : 0] = mul2(prod[CHANNEL ? 2 * i4 + 1 : 0], a4.y);
               }
             }
-            if (!LOCAL) {
-              const float4 q4 = *reinterpret_cast<const float4*>(row + Q_AT + (i4 * RL + rl) * 4);
-              qq[0] = q4.x; qq[1] = q4.y; qq[2] = q4.z; qq[3] = q4.w;
-            }
+            if (!LOCAL) q4 = *reinterpret_cast<const ulonglong2*>(row + Q_AT + (i4 * RL + rl) * 4);
 #pragma unroll
-            for (int e = 0; e < 4; e++)
-#pragma unroll
-              for (int c = 0; c < DC_TC; c++) {
-                float& x = s[i4 * 4 + e][c];
-                x = fmaf(CHANNEL ? aa[e] : ah, x, kk[e] * v[c]);
-                if (!LOCAL) acc[u * DC_TC + c] = fmaf(x, qq[e], acc[u * DC_TC + c]);
+            for (int c = 0; c < DC_TC; c++) {
+              s[2 * i4][c] = fma2(a4.x, s[2 * i4][c], mul2(k4.x, v2[c]));
+              s[2 * i4 + 1][c] = fma2(a4.y, s[2 * i4 + 1][c], mul2(k4.y, v2[c]));
+              if (!LOCAL) {
+                o2[c] = fma2(s[2 * i4][c], q4.x, o2[c]);
+                o2[c] = fma2(s[2 * i4 + 1][c], q4.y, o2[c]);
               }
+            }
+          }
+          if (!LOCAL) {
+#pragma unroll
+            for (int c = 0; c < DC_TC; c++) {
+              const float2 f = unpack2(o2[c]);
+              acc[u * DC_TC + c] += f.x + f.y;
+            }
           }
         }
       }
@@ -273,7 +292,10 @@ decay_recurrence_kernel(DecayRec p) {
             if (cg * DC_TC + c + i < cols_here) dst[i] = acc[i] * p.q_scale;
         }
       }
-    }
+    };
+    int tt = 0;
+    for (; tt + DC_NT <= nt; tt += DC_NT) four(tt, DcTrue{});
+    if (tt < nt) four(tt, DcFalse{});
   }
   asm volatile("cp.async.wait_group 0;\n" ::: "memory");
   float* S1;
@@ -284,28 +306,38 @@ decay_recurrence_kernel(DecayRec p) {
       if (cg == 0 && c0 == 0) {
         float* d = p.seg_decay + ((long long)seq * p.n_seg + seg) * p.n_heads * p.dim + h * p.dim + r0;
 #pragma unroll
-        for (int i = 0; i < DC_TR; i++) {
-          const int r = ((i >> 2) * RL + rl) * 4 + (i & 3);
-          if (r < rows_here) d[r] = prod[CHANNEL ? i : 0];
+        for (int i = 0; i < DC_TR / 2; i++) {
+          const int r = ((i >> 1) * RL + rl) * 4 + (i & 1) * 2;
+          const float2 f = unpack2(prod[CHANNEL ? i : 0]);
+          if (r < rows_here) d[r] = f.x;
+          if (r + 1 < rows_here) d[r + 1] = f.y;
         }
       }
     } else if (threadIdx.x == 0 && c0 == 0 && rg == 0) {
-      p.seg_decay[((long long)seq * p.n_seg + seg) * p.n_heads + h] = prod[0];
+      p.seg_decay[((long long)seq * p.n_seg + seg) * p.n_heads + h] = unpack2(prod[0]).x;
     }
   } else {
     if (seg != own_segs - 1) return;
     S1 = slot_state;
   }
 #pragma unroll
-  for (int i = 0; i < DC_TR; i++) {
-    const int r = ((i >> 2) * RL + rl) * 4 + (i & 3);
-    if (r < rows_here) {
-      if (p.vec && cg * DC_TC < cols_here) {
-        *reinterpret_cast<float4*>(S1 + (long long)r * p.vdim) = make_float4(s[i][0], s[i][1], s[i][2], s[i][3]);
-      } else {
+  for (int i = 0; i < DC_TR / 2; i++) {
+    float2 x[DC_TC];
 #pragma unroll
-        for (int c = 0; c < DC_TC; c++)
-          if (cg * DC_TC + c < cols_here) S1[(long long)r * p.vdim + c] = s[i][c];
+    for (int c = 0; c < DC_TC; c++) x[c] = unpack2(s[i][c]);
+#pragma unroll
+    for (int e = 0; e < 2; e++) {
+      const int r = ((i >> 1) * RL + rl) * 4 + (i & 1) * 2 + e;
+      if (r < rows_here) {
+        float* dst = S1 + (long long)r * p.vdim;
+        if (p.vec && cg * DC_TC < cols_here) {
+          *reinterpret_cast<float4*>(dst) = e ? make_float4(x[0].y, x[1].y, x[2].y, x[3].y)
+                                              : make_float4(x[0].x, x[1].x, x[2].x, x[3].x);
+        } else {
+#pragma unroll
+          for (int c = 0; c < DC_TC; c++)
+            if (cg * DC_TC + c < cols_here) dst[c] = e ? x[c].y : x[c].x;
+        }
       }
     }
   }
@@ -365,6 +397,42 @@ MF_API int mf_decay_blocks(int n_heads, int dim, int vdim) {
   const DcShape s = dc_shape(dim, vdim);
   return n_heads * mf_decay_parts(dim, vdim) * ((vdim + s.cg * DC_TC - 1) / (s.cg * DC_TC));
 }
+
+// Blocks of a launch that the GPU holds at a time (looked up once per device and shape).
+template <int RL, int CG, bool CHANNEL, bool LOCAL>
+static int dc_resident() {
+  static int n[MF_MAX_DEVICES] = {};
+  const int dev = mf_current_device();
+  if (dev < 0) return 0;
+  if (!n[dev]) {
+    constexpr int NA = (LOCAL ? 1 : 2) + (CHANNEL ? 1 : 0);
+    constexpr size_t smem = (size_t)DC_STAGES * DC_CHUNK * (NA * RL * DC_TR + CG * DC_TC + 4) * sizeof(float);
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(decay_recurrence_kernel<RL, CG, CHANNEL, LOCAL>,
+                                                 cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+      return 0;
+    int per = 0;
+    if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per, decay_recurrence_kernel<RL, CG, CHANNEL, LOCAL>, RL * CG, smem) !=
+        cudaSuccess)
+      return 0;
+    n[dev] = per * mf_sm_count();
+  }
+  return n[dev];
+}
+#define DC_RESIDENT(RL, CG)                                                                                 \
+  if (s.rl == RL && s.cg == CG)                                                                             \
+  return per_channel ? (local ? dc_resident<RL, CG, true, true>() : dc_resident<RL, CG, true, false>())     \
+                     : (local ? dc_resident<RL, CG, false, true>() : dc_resident<RL, CG, false, false>())
+MF_API int mf_decay_resident(int dim, int vdim, int per_channel, int local) {
+  const DcShape s = dc_shape(dim, vdim);
+  DC_RESIDENT(4, 8);
+  DC_RESIDENT(8, 8);
+  DC_RESIDENT(16, 8);
+  DC_RESIDENT(4, 16);
+  DC_RESIDENT(8, 16);
+  DC_RESIDENT(16, 16);
+  return 0;
+}
+#undef DC_RESIDENT
 
 template <int RL, int CG, bool CHANNEL, bool LOCAL>
 static int dc_launch(const DecayRec& p, int n_seqs, cudaStream_t stream) {

@@ -6,6 +6,7 @@ pointers and the current stream, and raise ``KernelError`` on a refusal.
 from __future__ import annotations
 
 from ctypes import c_void_p
+from functools import lru_cache
 from typing import Optional
 
 import torch
@@ -843,19 +844,35 @@ def conv_act(x: torch.Tensor, ld: int, w: torch.Tensor, bias: Optional[torch.Ten
           launches=2 if taps > 1 and T != batch.n_seqs else 1)
 
 
-SCAN_TARGET_BLOCKS = 888      # blocks a recurrence over a long portion is cut up for: six for every SM
+SCAN_LOCAL_COST = 0.6         # of a pass from a zero state, beside the pass with the read-outs
+SCAN_MAX_FLOATS = 64 << 20    # of start states (256 MB)
 
 
-def scan_segments(batch, blocks: int, state_floats: int, min_tokens: int, piece: int = 8):
-    """(number of segments, their length) into which a linear recurrence cuts the step's longest portion:
-    as many as fill the GPU beside the ``blocks`` blocks that a sequence has anyway, none shorter than
-    ``min_tokens``, within 256 MB of states; one segment where every portion is short."""
+@lru_cache(maxsize=4096)
+def _segment_count(blocks: int, resident: int, local: int, most: int) -> int:
+    """The number of segments with the least waves of blocks times their length: ``blocks`` for every segment,
+    ``resident`` of the last pass and ``local`` of the first at a time on the GPU."""
+    if resident < 1 or local < 1:
+        return 1
+    best, best_cost = 1, float(-(-blocks // resident))
+    for n in range(2, most + 1):
+        cost = (-(-n * blocks // resident) + SCAN_LOCAL_COST * -(-(n - 1) * blocks // local)) / n + 0.002 * n
+        if cost < best_cost - 1e-9:
+            best, best_cost = n, cost
+    return best
+
+
+def scan_segments(batch, blocks: int, residents, state_floats: int, min_tokens: int, piece: int = 8):
+    """(number of segments, their length) into which a linear recurrence cuts the step's longest portion: what
+    fills the GPU best beside the ``blocks`` blocks that a sequence has anyway, none shorter than
+    ``min_tokens``, within ``SCAN_MAX_FLOATS`` of states; one segment where every portion is short.
+    ``residents``: blocks of the last and of the first pass that the GPU holds at a time."""
     longest = max(batch.q_len)
     if longest < 2 * min_tokens:
         return 1, longest
     n_long = sum(1 for n in batch.q_len if n >= 2 * min_tokens)
-    n = min(-(-SCAN_TARGET_BLOCKS // (blocks * n_long)), longest // min_tokens,
-            max(1, (64 << 20) // (batch.n_seqs * state_floats)))
+    most = min(longest // min_tokens, max(1, SCAN_MAX_FLOATS // (batch.n_seqs * state_floats)), 256)
+    n = _segment_count(blocks * n_long, residents[0], residents[1], most)
     if n < 2:
         return 1, longest
     length = -(-longest // n)
@@ -871,6 +888,11 @@ def decay_parts(dim: int, vdim: int) -> int:
 def decay_blocks(n_heads: int, dim: int, vdim: int) -> int:
     """Blocks of ``decay_recurrence`` per sequence and segment."""
     return int(library().mf_decay_blocks(n_heads, dim, vdim))
+
+
+def decay_residents(dim: int, vdim: int, per_channel: bool):
+    """Blocks of ``decay_recurrence`` that the GPU holds at a time: of the pass with read-outs, of the one without."""
+    return tuple(int(library().mf_decay_resident(dim, vdim, int(per_channel), local)) for local in (0, 1))
 
 
 def decay_recurrence(q: torch.Tensor, q_ld: int, k: torch.Tensor, k_ld: int, v: torch.Tensor, v_ld: int,
@@ -918,6 +940,10 @@ def gated_norm(x: torch.Tensor, gate: torch.Tensor, gate_ld: int, weight: torch.
 def scan_blocks(channels: int, n_state: int) -> int:
     """Blocks of ``selective_scan`` per sequence and segment (0: more states than it takes)."""
     return int(library().mf_scan_blocks(channels, n_state))
+
+
+def scan_residents(n_state: int):
+    return tuple(int(library().mf_scan_resident(n_state, local)) for local in (0, 1))
 
 
 def selective_scan(u: torch.Tensor, dt: torch.Tensor, dt_ld: int, dt_bias: torch.Tensor, z: torch.Tensor, z_ld: int,

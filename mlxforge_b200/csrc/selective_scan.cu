@@ -25,6 +25,18 @@ constexpr int SS_THREADS = 128;
 constexpr int SS_CHUNK = 8;          // tokens per stage
 __device__ __forceinline__ float ss_softplus(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float ss_silu(float x) { return x / (1.0f + expf(-x)); }
+// FAST: the exponents were multiplied by log2 e and the special function unit's power of two (its relative error is
+// below 2^-22) is the decay; else expf.
+template <bool FAST>
+__device__ __forceinline__ float ss_exp(float x) {
+  if constexpr (FAST) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+  } else {
+    return expf(x);
+  }
+}
 }  // namespace
 
 struct ScanArgs {
@@ -48,7 +60,7 @@ struct ScanArgs {
   int seg_len, n_seg, channels, n_state;
 };
 
-template <typename TO, int LN, bool LOCAL>
+template <typename TO, int LN, bool LOCAL, bool FAST>
 __global__ void __launch_bounds__(SS_THREADS)
 selective_scan_kernel(ScanArgs p, TO* __restrict__ out) {
   constexpr int CB = SS_THREADS / LN;                        // channels of the block
@@ -74,14 +86,39 @@ selective_scan_kernel(ScanArgs p, TO* __restrict__ out) {
   const long long SSZ = (long long)p.channels * N;
   float* slot_state = p.state + (long long)p.slots[seq] * p.state_stride;
   const float* S0 = own_segs > 1 ? p.seg_state + ((long long)seq * p.n_seg + seg) * SSZ : slot_state;
-  // state i of a thread: ((i / 4) * LN + ln) * 4 + i % 4
-  float s[SS_NS], A[SS_NS];
+  // state i of a thread: ((i / 4) * LN + ln) * 4 + i % 4; states 2 i and 2 i + 1 stand in one register pair
+  f32x2 s[SS_NS / 2], A[SS_NS / 2];
+  const bool whole = (N & 3) == 0;                           // states come in pieces of 16 bytes
 #pragma unroll
-  for (int i = 0; i < SS_NS; i++) {
-    const int m = ((i >> 2) * LN + ln) * 4 + (i & 3);
-    const bool in = live && m < N;
-    A[i] = in ? p.A[(long long)c * N + m] : 0.f;
-    s[i] = (!LOCAL && in) ? S0[(long long)c * N + m] : 0.f;
+  for (int i4 = 0; i4 < SS_NS / 4; i4++) {
+    const int m = (i4 * LN + ln) * 4;
+    float a[4] = {0.f, 0.f, 0.f, 0.f}, x[4] = {0.f, 0.f, 0.f, 0.f};
+    if (live && m < N) {
+      const long long at = (long long)c * N + m;
+      if (whole) {
+        const float4 f = *reinterpret_cast<const float4*>(p.A + at);
+        a[0] = f.x; a[1] = f.y; a[2] = f.z; a[3] = f.w;
+        if (!LOCAL) {
+          const float4 g = *reinterpret_cast<const float4*>(S0 + at);
+          x[0] = g.x; x[1] = g.y; x[2] = g.z; x[3] = g.w;
+        }
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; e++)
+          if (m + e < N) {
+            a[e] = p.A[at + e];
+            if (!LOCAL) x[e] = S0[at + e];
+          }
+      }
+    }
+    if (FAST) {
+#pragma unroll
+      for (int e = 0; e < 4; e++) a[e] *= 1.4426950408889634f;
+    }
+    A[2 * i4] = pack2(a[0], a[1]);
+    A[2 * i4 + 1] = pack2(a[2], a[3]);
+    s[2 * i4] = pack2(x[0], x[1]);
+    s[2 * i4 + 1] = pack2(x[2], x[3]);
   }
   // operands of the coming run: this thread's (token, channel) items, fetched into registers a run ahead
   float rdt[ITEMS], ru[ITEMS], rz[ITEMS];
@@ -144,23 +181,22 @@ selective_scan_kernel(ScanArgs p, TO* __restrict__ out) {
     for (int tok = 0; tok < nt; tok++) {
       const float4 w = o4[tok * CB + cl];
       const float* B = bcs + tok * 2 * NP;
-      float y = 0.f;
+      const f32x2 dt2 = pack2(w.x, w.x), du2 = pack2(w.y, w.y);
+      f32x2 y2 = 0;
 #pragma unroll
       for (int i4 = 0; i4 < SS_NS / 4; i4++) {
-        const float4 b4 = *reinterpret_cast<const float4*>(B + (i4 * LN + ln) * 4);
-        const float b[4] = {b4.x, b4.y, b4.z, b4.w};
-        float cc[4];
+        const ulonglong2 b4 = *reinterpret_cast<const ulonglong2*>(B + (i4 * LN + ln) * 4);
+        const float2 e0 = unpack2(mul2(dt2, A[2 * i4])), e1 = unpack2(mul2(dt2, A[2 * i4 + 1]));
+        s[2 * i4] = fma2(pack2(ss_exp<FAST>(e0.x), ss_exp<FAST>(e0.y)), s[2 * i4], mul2(du2, b4.x));
+        s[2 * i4 + 1] = fma2(pack2(ss_exp<FAST>(e1.x), ss_exp<FAST>(e1.y)), s[2 * i4 + 1], mul2(du2, b4.y));
         if (!LOCAL) {
-          const float4 c4 = *reinterpret_cast<const float4*>(B + NP + (i4 * LN + ln) * 4);
-          cc[0] = c4.x; cc[1] = c4.y; cc[2] = c4.z; cc[3] = c4.w;
-        }
-#pragma unroll
-        for (int e = 0; e < 4; e++) {
-          float& x = s[i4 * 4 + e];
-          x = fmaf(expf(w.x * A[i4 * 4 + e]), x, w.y * b[e]);
-          if (!LOCAL) y = fmaf(x, cc[e], y);
+          const ulonglong2 c4 = *reinterpret_cast<const ulonglong2*>(B + NP + (i4 * LN + ln) * 4);
+          y2 = fma2(s[2 * i4], c4.x, y2);
+          y2 = fma2(s[2 * i4 + 1], c4.y, y2);
         }
       }
+      const float2 yy = unpack2(y2);
+      float y = yy.x + yy.y;
       if (LOCAL) {
         dt_sum += w.x;
       } else {
@@ -180,9 +216,20 @@ selective_scan_kernel(ScanArgs p, TO* __restrict__ out) {
     S1 = slot_state;
   }
 #pragma unroll
-  for (int i = 0; i < SS_NS; i++) {
-    const int m = ((i >> 2) * LN + ln) * 4 + (i & 3);
-    if (live && m < N) S1[(long long)c * N + m] = s[i];
+  for (int i4 = 0; i4 < SS_NS / 4; i4++) {
+    const int m = (i4 * LN + ln) * 4;
+    if (live && m < N) {
+      float* dst = S1 + (long long)c * N + m;
+      const float2 x0 = unpack2(s[2 * i4]), x1 = unpack2(s[2 * i4 + 1]);
+      if (whole) {
+        *reinterpret_cast<float4*>(dst) = make_float4(x0.x, x0.y, x1.x, x1.y);
+      } else {
+        dst[0] = x0.x;
+        if (m + 1 < N) dst[1] = x0.y;
+        if (m + 2 < N) dst[2] = x1.x;
+        if (m + 3 < N) dst[3] = x1.y;
+      }
+    }
   }
 }
 
@@ -236,34 +283,56 @@ MF_API int mf_scan_blocks(int channels, int n_state) {
   return (channels + cb - 1) / cb;
 }
 
-template <typename TO, int LN, bool LOCAL>
-static int ss_launch(const ScanArgs& p, void* out, int n_seqs, cudaStream_t stream) {
-  constexpr int CB = SS_THREADS / LN;
-  constexpr size_t smem = (size_t)(2 * SS_CHUNK * CB * 4 + 2 * SS_CHUNK * 2 * LN * SS_NS) * sizeof(float);
-  static DeviceOnce once;
-  const int dev = mf_current_device();
-  if (dev < 0) return MF_ERR_BAD_ARG;
-  if (!once.done[dev] && smem > 48 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(selective_scan_kernel<TO, LN, LOCAL>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                         (int)smem);
-    if (e != cudaSuccess) return (int)e;
+template <typename TO, int LN, bool LOCAL, bool FAST>
+struct SsKernel {
+  static constexpr int CB = SS_THREADS / LN;
+  static constexpr size_t smem = (size_t)(2 * SS_CHUNK * CB * 4 + 2 * SS_CHUNK * 2 * LN * SS_NS) * sizeof(float);
+  // blocks that the GPU holds at a time (looked up once per device); 0: it cannot run
+  static int resident() {
+    static int n[MF_MAX_DEVICES] = {};
+    const int dev = mf_current_device();
+    if (dev < 0) return 0;
+    if (!n[dev]) {
+      if (smem > 48 * 1024 && cudaFuncSetAttribute(selective_scan_kernel<TO, LN, LOCAL, FAST>,
+                                                   cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+        return 0;
+      int per = 0;
+      if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per, selective_scan_kernel<TO, LN, LOCAL, FAST>, SS_THREADS, smem) !=
+          cudaSuccess)
+        return 0;
+      n[dev] = per * mf_sm_count();
+    }
+    return n[dev];
   }
-  once.done[dev] = true;
-  return (int)launch_dep(selective_scan_kernel<TO, LN, LOCAL>, dim3(n_seqs, (p.channels + CB - 1) / CB, p.n_seg),
-                         dim3(SS_THREADS), smem, stream, p, (TO*)out);
-}
+  static int launch(const ScanArgs& p, void* out, int n_seqs, cudaStream_t stream) {
+    if (resident() <= 0) return MF_ERR_BAD_ARG;
+    return (int)launch_dep(selective_scan_kernel<TO, LN, LOCAL, FAST>, dim3(n_seqs, (p.channels + CB - 1) / CB, p.n_seg),
+                           dim3(SS_THREADS), smem, stream, p, (TO*)out);
+  }
+};
+#define SS_BY_LANES(n_state, TO, LOCAL, FAST, CALL)             \
+  switch (ss_lanes(n_state)) {                                  \
+    case 1: return SsKernel<TO, 1, LOCAL, FAST>::CALL;          \
+    case 2: return SsKernel<TO, 2, LOCAL, FAST>::CALL;          \
+    case 4: return SsKernel<TO, 4, LOCAL, FAST>::CALL;          \
+    case 8: return SsKernel<TO, 8, LOCAL, FAST>::CALL;          \
+    case 16: return SsKernel<TO, 16, LOCAL, FAST>::CALL;        \
+    case 32: return SsKernel<TO, 32, LOCAL, FAST>::CALL;        \
+  }
 
-template <typename TO, bool LOCAL>
+template <typename TO, bool LOCAL, bool FAST>
 static int ss_pick(const ScanArgs& p, void* out, int n_seqs, cudaStream_t stream) {
-  switch (ss_lanes(p.n_state)) {
-    case 1: return ss_launch<TO, 1, LOCAL>(p, out, n_seqs, stream);
-    case 2: return ss_launch<TO, 2, LOCAL>(p, out, n_seqs, stream);
-    case 4: return ss_launch<TO, 4, LOCAL>(p, out, n_seqs, stream);
-    case 8: return ss_launch<TO, 8, LOCAL>(p, out, n_seqs, stream);
-    case 16: return ss_launch<TO, 16, LOCAL>(p, out, n_seqs, stream);
-    case 32: return ss_launch<TO, 32, LOCAL>(p, out, n_seqs, stream);
-  }
+  SS_BY_LANES(p.n_state, TO, LOCAL, FAST, launch(p, out, n_seqs, stream))
   return MF_ERR_BAD_ARG;
+}
+template <typename TO, bool LOCAL, bool FAST>
+static int ss_resident(int n_state) {
+  SS_BY_LANES(n_state, TO, LOCAL, FAST, resident())
+  return 0;
+}
+// Blocks that the GPU holds at a time, of the serving (bfloat16) form; `local`: of the pass from a zero state.
+MF_API int mf_scan_resident(int n_state, int local) {
+  return local ? ss_resident<float, true, true>(n_state) : ss_resident<__nv_bfloat16, false, true>(n_state);
 }
 
 MF_API int mf_selective_scan(const float* u, const float* dt, int dt_ld, const float* dt_bias, const float* z, int z_ld,
@@ -275,12 +344,16 @@ MF_API int mf_selective_scan(const float* u, const float* dt, int dt_ld, const f
   const int blocks = n_state > 0 && channels > 0 ? mf_scan_blocks(channels, n_state) : 0;
   if (blocks < 1 || blocks > 65535 || seg_len <= 0 || n_seg < 1 || n_seg > 65535) return MF_ERR_BAD_ARG;
   if (n_seg > 1 && (!seg_state || !seg_dt)) return MF_ERR_BAD_ARG;
+  // states in pieces of 16 bytes are read so
+  if (n_state % 4 == 0 && (((uintptr_t)state | (uintptr_t)A | (uintptr_t)seg_state) & 15 || state_stride % 4))
+    return MF_ERR_BAD_ARG;
   if (out_dtype != MF_F32 && out_dtype != MF_BF16) return MF_ERR_BAD_DTYPE;
   const ScanArgs p{u, dt, dt_ld, dt_bias, z, z_ld, bc, bc_ld, A, D, state, state_stride, seq_q_start, seq_q_len, slots,
                    seg_state, seg_dt, seg_len, n_seg, channels, n_state};
   if (n_seg > 1) {
     mf_count(MF_K_SCAN_LOCAL);
-    int e = ss_pick<float, true>(p, nullptr, n_seqs, stream);
+    int e = out_dtype == MF_F32 ? ss_pick<float, true, false>(p, nullptr, n_seqs, stream)
+                                : ss_pick<float, true, true>(p, nullptr, n_seqs, stream);
     if (e) return e;
     const long long SSZ = (long long)channels * n_state;
     mf_count(MF_K_SCAN_COMBINE);
@@ -290,8 +363,8 @@ MF_API int mf_selective_scan(const float* u, const float* dt, int dt_ld, const f
     if (e) return e;
   }
   mf_count(MF_K_SELECTIVE_SCAN);
-  return out_dtype == MF_F32 ? ss_pick<float, false>(p, out, n_seqs, stream)
-                             : ss_pick<__nv_bfloat16, false>(p, out, n_seqs, stream);
+  return out_dtype == MF_F32 ? ss_pick<float, false, false>(p, out, n_seqs, stream)
+                             : ss_pick<__nv_bfloat16, false, true>(p, out, n_seqs, stream);
 }
 
 // ------------------------------------------------------------------ a narrow product and what follows it
@@ -301,6 +374,7 @@ MF_API int mf_selective_scan(const float* u, const float* dt, int dt_ld, const f
 // tokens of its own and the block's weights lie in shared memory.
 namespace {
 constexpr int LR_TOK = 8;
+constexpr int LR_PIECE = 128;        // of the rank, at a time
 __device__ __forceinline__ float lr_act(float x, int f, float inv_tau) {
   if (f == 0) return x;
   const float nx = -x;
@@ -313,22 +387,33 @@ __global__ void __launch_bounds__(256)
 low_rank_split_kernel(const float* __restrict__ low, int ld, const TW* __restrict__ wt, const float* __restrict__ bias,
                       int f, float inv_tau, float* __restrict__ out, int T, int R, int n) {
   __shared__ float part[8][LR_TOK][32];
+  __shared__ float ls[LR_TOK][LR_PIECE];
   pdl_launch();
-  pdl_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int j = blockIdx.x * 32 + lane, t0 = blockIdx.y * LR_TOK;
   const int nt = min(LR_TOK, T - t0);
   float acc[LR_TOK];
 #pragma unroll
   for (int u = 0; u < LR_TOK; u++) acc[u] = 0.f;
-  if (j < n) {
-#pragma unroll 4
-    for (int r = warp; r < R; r += 8) {
-      const float w = to_f32<TW>(wt[(long long)r * n + j]);
+  for (int r0 = 0; r0 < R; r0 += LR_PIECE) {
+    const int nr = min(LR_PIECE, R - r0);
+    float w[LR_PIECE / 8];          // the weights never change: the first piece's are fetched before the wait
 #pragma unroll
-      for (int u = 0; u < LR_TOK; u++)
-        if (u < nt) acc[u] = fmaf(w, low[(long long)(t0 + u) * ld + r], acc[u]);
+    for (int q = 0; q < LR_PIECE / 8; q++) {
+      const int r = q * 8 + warp;
+      w[q] = (r < nr && j < n) ? to_f32<TW>(wt[(long long)(r0 + r) * n + j]) : 0.f;
     }
+    if (r0 == 0) pdl_wait();
+    else __syncthreads();
+    for (int i = threadIdx.x; i < LR_TOK * LR_PIECE; i += 256) {
+      const int u = i / LR_PIECE, r = i - u * LR_PIECE;
+      ls[u][r] = (u < nt && r < nr) ? low[(long long)(t0 + u) * ld + r0 + r] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int q = 0; q < LR_PIECE / 8; q++)
+#pragma unroll
+      for (int u = 0; u < LR_TOK; u++) acc[u] = fmaf(w[q], ls[u][q * 8 + warp], acc[u]);
   }
 #pragma unroll
   for (int u = 0; u < LR_TOK; u++) part[warp][u][lane] = acc[u];

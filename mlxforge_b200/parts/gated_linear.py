@@ -72,7 +72,7 @@ class GatedLinear(_Scan):
         alpha = rt.buffer("gla.alpha", (T, nqk), f32)
         ops.low_rank(proj[:, 2 * nqk + 2 * nv:], ld, self.w_a2_t, self.a_bias, alpha, decay_tau=self.tau)
         o = self._readouts(T, ops.decay_parts(d, dv), nv)
-        seg, scratch = self._segments(batch, ops.decay_blocks(nh, d, dv), self.state_floats, nqk)
+        seg, scratch = self._segments(batch, ops.decay_blocks(nh, d, dv), ops.decay_residents(d, dv, True), self.state_floats, nqk)
         ops.decay_recurrence(proj, ld, proj[:, nqk:], ld, proj[:, 2 * nqk:], ld, cache.tensor, batch, o, nh, nh, d, dv,
                              alpha=alpha, q_scale=self.q_scale, segments=seg, scratch=scratch)
         y = rt.buffer("scan.y", (T, nv))

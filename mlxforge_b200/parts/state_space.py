@@ -56,8 +56,8 @@ class _Scan(Mixer):
     def _n(self, role: str) -> str:
         return self.prefix + self.names[role]
 
-    def _segments(self, batch, blocks: int, state_floats: int, decay_floats: int):
-        seg = ops.scan_segments(batch, blocks, state_floats, self.min_tokens)
+    def _segments(self, batch, blocks: int, residents, state_floats: int, decay_floats: int):
+        seg = ops.scan_segments(batch, blocks, residents, state_floats, self.min_tokens)
         if seg[0] == 1:
             return seg, None
         n = batch.n_seqs * seg[0]
@@ -132,8 +132,8 @@ class Mamba2(_Scan):
         xbc = rt.buffer("mamba2.xbc", (T, self.channels), f32)
         ops.conv_act(proj[:, self.inner:], ld, self.conv_w, self.conv_b, True, cache.tensor, self.conv_off, batch, xbc)
         o = self._readouts(T, ops.decay_parts(self.state, self.vdim), self.inner)
-        seg, scratch = self._segments(batch, ops.decay_blocks(self.n_heads, self.state, self.vdim), self.state_floats,
-                                      self.n_heads)
+        seg, scratch = self._segments(batch, ops.decay_blocks(self.n_heads, self.state, self.vdim),
+                                      ops.decay_residents(self.state, self.vdim, False), self.state_floats, self.n_heads)
         C = self.channels
         ops.decay_recurrence(xbc[:, self.inner + self.bc:], C, xbc[:, self.inner:], C, xbc, C, cache.tensor, batch, o,
                              self.n_heads, self.groups, self.state, self.vdim, dt=proj[:, self.inner + C:], dt_ld=ld,
@@ -202,7 +202,7 @@ class SelectiveScan(_Scan):
             rt.linear(dt_low, self.w_dt, dt)
         else:
             ops.low_rank(low, low.shape[1], self.w_dt_t, None, dt)
-        seg, scratch = self._segments(batch, ops.scan_blocks(n, self.state), self.state_floats, n)
+        seg, scratch = self._segments(batch, ops.scan_blocks(n, self.state), ops.scan_residents(self.state), self.state_floats, n)
         y = rt.buffer("sscan.y", (T, n))
         ops.selective_scan(u, dt, n, self.dt_bias, proj[:, n:], 2 * n, low[:, R:], low.shape[1], self.a, self.d,
                            cache.tensor, batch, y, self.state, seg, scratch)

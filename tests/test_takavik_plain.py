@@ -228,17 +228,18 @@ def test_cache_layout_pages_beside_states():
 
 
 def test_how_a_portion_is_cut_into_segments():
-    from mlxforge_b200.csrc.ops import SCAN_TARGET_BLOCKS, scan_segments
+    from mlxforge_b200.csrc.ops import SCAN_MAX_FLOATS, scan_segments
     b = lambda *lens: SimpleNamespace(q_len=list(lens), n_seqs=len(lens))
-    assert scan_segments(b(1, 1, 1), 4, 1000, 64) == (1, 1)           # a decode step runs in one piece
-    assert scan_segments(b(127, 1), 4, 1000, 64) == (1, 127)
+    held = (300, 600)
+    assert scan_segments(b(1, 1, 1), 4, held, 1000, 64) == (1, 1)     # a decode step runs in one piece
+    assert scan_segments(b(127, 1), 4, held, 1000, 64) == (1, 127)
     for lens, blocks, least in (((2048,), 32, 64), ((300, 1, 129), 3, 64), ((45, 23), 2, 8), ((1000,), 100, 64)):
-        n, length = scan_segments(b(*lens), blocks, 1000, least)
+        n, length = scan_segments(b(*lens), blocks, held, 1000, least)
         assert n > 1 and n * length >= max(lens) > (n - 1) * length and length % 8 == 0 and length >= least
-        assert n * blocks <= SCAN_TARGET_BLOCKS + blocks
-    assert scan_segments(b(2048), SCAN_TARGET_BLOCKS, 1000, 64) == (1, 2048)      # the GPU is full without
-    n, _ = scan_segments(b(4096), 1, 8 << 20, 64)
-    assert n <= 8                                                     # within 64 million numbers of scratch
+    assert scan_segments(b(2048), 300, held, 1000, 64) == (1, 2048)   # the GPU is full without
+    assert scan_segments(b(2048), 4, (0, 0), 1000, 64) == (1, 2048)   # how full it is cannot be had
+    n, _ = scan_segments(b(4096), 1, held, SCAN_MAX_FLOATS // 8, 64)
+    assert n <= 8                                                     # within the scratch for start states
 
 
 def test_configurations_drawn_at_random_are_read():
