@@ -94,7 +94,6 @@ class Mamba2(_Scan):
             raise ValueError("mamba2: conv must be at least 1 tap")
         self.state_floats = self.n_heads * self.state * self.vdim
         self.conv_off = pad4(self.state_floats)
-        # rows of the projection are padded to whole pieces of 16 bytes
         self.width = self.inner + self.channels + self.n_heads
         self.w_in = self.w_o = self.conv_w = self.conv_b = self.dt_bias = self.a_log = self.d = self.norm_w = None
 
@@ -111,7 +110,7 @@ class Mamba2(_Scan):
         dt, f32 = self.rt.dtype, torch.float32
         w = tensors[self._n("in")].to(dt)
         pad = pad4(self.width) - self.width
-        if pad:
+        if pad:                                    # rows of the projection in whole pieces of 16 bytes
             w = torch.cat([w, torch.zeros((pad, self.hidden), dtype=dt, device=w.device)], dim=0)
         self.w_in = w.contiguous()
         self.w_o = tensors[self._n("o")].to(dt).contiguous()

@@ -112,7 +112,7 @@ ATTN_CASES = {
     "ones": (1, 1, 16, 16, 0.0, 1),
     "every_token": (2, 2, 8, 8, 0.4, 1),
     "tc64": (4, 2, 64, 64, 0.5, 33),
-    "tc96": (8, 2, 96, 96, 0.5, 64),
+    "tc96": (6, 3, 96, 96, 0.4, 40),
     "tc128": (4, 1, 128, 128, 0.3, 50),
     "tc128v64": (4, 2, 128, 64, 0.3, 50),
     "wide_values": (2, 1, 48, 80, 0.3, 50),
