@@ -33,10 +33,10 @@ _SIGNATURES = {
     "mf_set_decode_status": [_P],
     "mf_set_decode_merge_inside": [c_int],
     "mf_attention_decode_launches": [],
-    "mf_gemm_bf16": [_P, _P, _P, c_int, c_int, c_int, c_int, _P, _P],
+    "mf_gemm_bf16": [_P, _P, _P, c_int, c_int, c_int, c_int, c_float, c_float, c_float, _P, _P],
     "mf_stream_max_rows": [],
     "mf_set_stream_tensor_copies": [c_int],
-    "mf_stream_linear": [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, _P],
+    "mf_stream_linear": [_P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float, _P, _P],
     "mf_attention_prefill": [_P, _P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, _P, c_int,
                              c_int, c_float, c_int, _P, _P],
     "mf_set_prefill_tcgen05": [c_int],
@@ -75,7 +75,7 @@ _SIGNATURES = {
     "mf_qk_norm_rope": [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, _P, _P, _P,
                         _P, _P, _P, _P, c_int, c_float, c_double, _P, _P, _P, c_int, c_int, _P, _P, _P, c_int, _P],
     "mf_rotate_rows": [_P, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, c_float, _P],
-    "mf_moe_route": [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P, _P, _P, _P],
+    "mf_moe_route": [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, _P, _P, _P, _P, _P],
     "mf_moe_rows": [_P, _P, _P, c_int, _P, _P, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_int, c_int, _P],
     "mf_moe_combine": [_P, c_int, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, c_int, _P, _P, _P, c_int, _P],
     "mf_moe_gather_rows": [_P, _P, _P, c_int, c_int, _P],
@@ -98,7 +98,12 @@ _SIGNATURES = {
                                 c_float, c_int, c_int, c_int, c_int, _P, _P, c_longlong, c_float, _P],
     "mf_attention_decode_ex": [_P, _P, _P, _P, _P, _P, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, c_int,
                                c_float, c_int, c_int, c_int, c_int, c_int, _P, _P, c_longlong, c_float, _P],
-    "mf_gated_act": [_P, _P, c_int, c_int, c_int, c_int, c_int, _P],
+    "mf_gated_act": [_P, _P, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, _P],
+    "mf_soft_cap": [_P, c_longlong, c_float, _P],
+    "mf_post_norm": [_P, _P, c_int, _P, c_int, c_float, _P, c_int, c_float, _P, c_int, _P, c_int, c_int, _P],
+    "mf_qkv_conv_ok": [c_int, c_int, c_int, c_int, c_int],
+    "mf_qkv_conv": [_P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, _P, c_int, _P, _P, _P, _P, _P,
+                    c_longlong, c_longlong, _P, _P, _P, _P, _P, c_int, _P, c_int, c_int, _P, _P, _P, _P],
     "mf_add_rmsnorm_pair": [_P, _P, _P, c_int, _P, _P, c_float, _P, _P, c_int, _P, c_int, c_int, _P],
     "mf_attention_generic_ex": [_P, _P, _P, _P, c_int, c_int, c_int, c_int, c_int, _P, _P, _P, c_int, c_int,
                                 c_float, c_int, c_int, c_int, c_int, _P, _P, c_int, c_float, _P],

@@ -43,6 +43,26 @@ __device__ __forceinline__ float gate_act(float g, int act) {
   return g / (1.0f + expf(-g));
 }
 
+// The clamped gate: g' = min(g, limit), u' = clamp(u, -limit, limit), g' sigmoid(alpha g') (u' + up_off).
+// It stands beside the activations above wherever a gate and an up value meet (not where there is no gate).
+#define MF_GATE_CLAMPED 8
+// mode of a product whose epilogue applies a soft cap to every sum: cap tanh(sum / cap)
+#define MF_STREAM_SOFTCAP 32
+// constants of a product's epilogue
+struct EpiConst {
+  float limit, alpha, up_off;      // of the clamped gate
+  float cap;                       // of the soft cap
+};
+__device__ __forceinline__ float gated_product(float g, float u, int act, const EpiConst& k) {
+  if (act == MF_GATE_CLAMPED) {
+    g = fminf(g, k.limit);
+    u = fminf(fmaxf(u, -k.limit), k.limit);
+    return g / (1.0f + expf(-k.alpha * g)) * (u + k.up_off);
+  }
+  return gate_act(g, act) * u;
+}
+__device__ __forceinline__ float soft_cap(float v, float cap) { return cap * tanhf(v / cap); }
+
 // Two 32-bit numbers side by side in a 64-bit register and the arithmetic on both at once (one instruction each,
 // rounded like the single ones).
 typedef unsigned long long f32x2;
@@ -242,6 +262,9 @@ enum MfKernel {
   MF_K_SELECTIVE_SCAN,        // a state per channel with token-dependent decay and input weights
   MF_K_SCAN_LOCAL,            // the same over segments from a zero state
   MF_K_LOW_RANK,              // a product with a narrow operand and the decay made of it
+  MF_K_POST_NORM,             // a sublayer's output through a norm of its own into the stream, and the stream's next norm
+  MF_K_QKV_CONV,              // convolved projections: norm per head, rotation, the cache write
+  MF_K_SOFT_CAP,              // cap tanh(x / cap) on rows of logits
   MF_K_COUNT
 };
 extern unsigned long long g_mf_kernel_launches[MF_K_COUNT];

@@ -9,7 +9,7 @@
 // however the tokens were cut; a second kernel moves them on after the first has read them.  Where
 // every sequence of the step brings one token a token's threads are the only readers of the slot's
 // rows and move them on themselves: one launch.
-#include "common.cuh"
+#include "conv_tail.cuh"
 
 __device__ __forceinline__ float ca_act(float v, int silu) { return silu ? v / (1.0f + expf(-v)) : v; }
 
@@ -131,6 +131,13 @@ conv_act_tail_kernel(const float* __restrict__ x, int ld, int C, int taps, float
     }
 }
 
+cudaError_t conv_tail_launch(const float* x, int ld, int C, int taps, float* state, long long state_stride,
+                             long long tail_off, const int* seq_q_start, const int* seq_q_len, const int* slots, int n_seqs,
+                             cudaStream_t stream) {
+  return launch_dep(conv_act_tail_kernel, dim3(n_seqs, (C + 1023) / 1024), dim3(256), 0, stream, x, ld, C, taps, state,
+                    state_stride, tail_off, seq_q_start, seq_q_len, slots);
+}
+
 MF_API int mf_conv_act(const float* x, int ld, int T, int C, const float* w, const float* bias, int taps, int silu,
                        float* state, long long state_stride, long long tail_off, const int* seq_of_token,
                        const int* seq_q_start, const int* seq_q_len, const int* slots, int n_seqs, float* out,
@@ -166,6 +173,5 @@ MF_API int mf_conv_act(const float* x, int ld, int T, int C, const float* w, con
 #undef CA_ANY
 #undef CA_VEC
   if (e != cudaSuccess || taps == 1 || single) return (int)e;
-  return (int)launch_dep(conv_act_tail_kernel, dim3(n_seqs, (C + 1023) / 1024), dim3(256), 0, stream, x, ld, C, taps,
-                         state, state_stride, tail_off, seq_q_start, seq_q_len, slots);
+  return (int)conv_tail_launch(x, ld, C, taps, state, state_stride, tail_off, seq_q_start, seq_q_len, slots, n_seqs, stream);
 }

@@ -332,9 +332,11 @@ MF_API int mf_rope_kv_write(const void* qkv, int dtype, int T, int n_heads, int 
 // gu [T, 2I] holds gate and up interleaved in groups of `group` columns:
 // gate i is column (i / group) * 2 * group + i % group, up i is `group` further.
 // group == I is the plain [gate | up] concatenation.  out[t, i] = act(gate) * up with
-// act = SiLU (MF_ACT_SILU) or the tanh form of GELU (MF_ACT_GELU_TANH), in 32-bit.
+// act = SiLU (MF_ACT_SILU) or the tanh form of GELU (MF_ACT_GELU_TANH), in 32-bit; MF_GATE_CLAMPED: the
+// clamped gate with its constants.
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, long long n, int I, int group, int act) {
+__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, long long n, int I, int group, int act,
+                              EpiConst ec) {
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= n) return;
   const long long t = idx / I;
@@ -342,12 +344,12 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, lon
   const int col = (i / group) * 2 * group + (i % group);
   const T* row = gu + t * 2 * (long long)I;
   const float g = to_f32<T>(row[col]), u = to_f32<T>(row[col + group]);
-  out[idx] = from_f32<T>(gate_act(g, act) * u);
+  out[idx] = from_f32<T>(gated_product(g, u, act, ec));
 }
 
 // bfloat16 with groups of 8: 16 bytes of gate, 16 bytes of up, 16 bytes out per thread
 __global__ void swiglu_bf16_g8_kernel(const uint4* __restrict__ gu, uint4* __restrict__ out, long long n_groups,
-                                      int act) {
+                                      int act, EpiConst ec) {
   const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= n_groups) return;
   const uint4 gv = gu[2 * idx], uv = gu[2 * idx + 1];
@@ -358,29 +360,30 @@ __global__ void swiglu_bf16_g8_kernel(const uint4* __restrict__ gu, uint4* __res
 #pragma unroll
   for (int e = 0; e < 4; e++) {
     const float2 g = __bfloat1622float2(gp[e]), u = __bfloat1622float2(up[e]);
-    p[e] = __floats2bfloat162_rn(gate_act(g.x, act) * u.x, gate_act(g.y, act) * u.y);
+    p[e] = __floats2bfloat162_rn(gated_product(g.x, u.x, act, ec), gated_product(g.y, u.y, act, ec));
   }
   out[idx] = pk;
 }
 
-MF_API int mf_gated_act(const void* gu, void* out, int dtype, int T, int I, int group, int act,
-                        cudaStream_t stream) {
+MF_API int mf_gated_act(const void* gu, void* out, int dtype, int T, int I, int group, int act, float limit,
+                        float alpha, float up_off, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (group <= 0 || I % group || act < 0 || act >= MF_ACT_COUNT) return MF_ERR_BAD_ARG;
+  if (group <= 0 || I % group || act < 0 || (act >= MF_ACT_COUNT && act != MF_GATE_CLAMPED)) return MF_ERR_BAD_ARG;
+  const EpiConst ec{limit, alpha, up_off, 0.f};
   if (dtype == MF_BF16 && group == 8 && (((uintptr_t)gu | (uintptr_t)out) & 15) == 0) {
     const long long n_groups = (long long)T * (I / 8);
     swiglu_bf16_g8_kernel<<<(unsigned)((n_groups + 255) / 256), 256, 0, stream>>>((const uint4*)gu, (uint4*)out,
-                                                                                    n_groups, act);
+                                                                                    n_groups, act, ec);
     return (int)cudaGetLastError();
   }
   const long long n = (long long)T * I;
   const int threads = 256;
   const unsigned blocks = (unsigned)((n + threads - 1) / threads);
   if (dtype == MF_F32)
-    swiglu_kernel<float><<<blocks, threads, 0, stream>>>((const float*)gu, (float*)out, n, I, group, act);
+    swiglu_kernel<float><<<blocks, threads, 0, stream>>>((const float*)gu, (float*)out, n, I, group, act, ec);
   else if (dtype == MF_BF16)
     swiglu_kernel<__nv_bfloat16><<<blocks, threads, 0, stream>>>((const __nv_bfloat16*)gu, (__nv_bfloat16*)out,
-                                                                 n, I, group, act);
+                                                                 n, I, group, act, ec);
   else
     return MF_ERR_BAD_DTYPE;
   return (int)cudaGetLastError();
@@ -433,7 +436,7 @@ MF_API int mf_unary_act(const void* in, void* out, int dtype, long long n, int a
 }
 
 MF_API int mf_swiglu(const void* gu, void* out, int dtype, int T, int I, int group, cudaStream_t stream) {
-  return mf_gated_act(gu, out, dtype, T, I, group, MF_ACT_SILU, stream);
+  return mf_gated_act(gu, out, dtype, T, I, group, MF_ACT_SILU, 0.f, 1.f, 0.f, stream);
 }
 
 // ------------------------------------------------------------------ add + two RMSNorms of one sum
@@ -586,6 +589,41 @@ MF_API int mf_add_rmsnorm_pair(float* resid, const void* d1, const void* d2, int
   if (delta_dtype == MF_BF16 && out_dtype == MF_F32) LAUNCH(__nv_bfloat16, float);
 #undef LAUNCH
   return MF_ERR_BAD_DTYPE;
+}
+
+// ------------------------------------------------------------------ soft cap
+// x[i] = cap tanh(x[i] / cap), in place, 32-bit (logits that a library product wrote)
+__global__ void __launch_bounds__(256) soft_cap_kernel(float* __restrict__ x, long long n, float cap) {
+  pdl_launch();
+  pdl_wait();
+  const long long step = (long long)gridDim.x * blockDim.x;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += step) x[i] = soft_cap(x[i], cap);
+}
+
+__global__ void __launch_bounds__(256) soft_cap_vec_kernel(float4* __restrict__ x, long long n4, float cap) {
+  pdl_launch();
+  pdl_wait();
+  const long long step = (long long)gridDim.x * blockDim.x;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < n4; i += step) {
+    float4 v = x[i];
+    v.x = soft_cap(v.x, cap);
+    v.y = soft_cap(v.y, cap);
+    v.z = soft_cap(v.z, cap);
+    v.w = soft_cap(v.w, cap);
+    x[i] = v;
+  }
+}
+
+MF_API int mf_soft_cap(float* x, long long n, float cap, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (!(cap > 0.f)) return MF_ERR_BAD_ARG;
+  mf_count(MF_K_SOFT_CAP);
+  const bool vec = n % 4 == 0 && ((uintptr_t)x & 15) == 0;
+  const long long items = vec ? n / 4 : n;
+  const long long blocks = (items + 255) / 256;
+  const dim3 grid((unsigned)(blocks < 148 * 8 ? blocks : 148 * 8));
+  if (vec) return (int)launch_dep(soft_cap_vec_kernel, grid, dim3(256), 0, stream, (float4*)x, items, cap);
+  return (int)launch_dep(soft_cap_kernel, grid, dim3(256), 0, stream, x, items, cap);
 }
 
 // ------------------------------------------------------------------ plain residual add

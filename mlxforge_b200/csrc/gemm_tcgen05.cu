@@ -89,18 +89,24 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<unsigned*>(&v);
 }
-template <int ACT> __device__ __forceinline__ float act_mul(float g, float u) { return gate_act(g, ACT) * u; }
+// the gate of an epilogue that multiplies gate and up
+constexpr int EPI_CLAMPED = 4 + MF_ACT_COUNT;
+template <int EPI> __device__ __forceinline__ float epi_gate(float g, float u, const EpiConst& ec) {
+  constexpr int act = EPI == EPI_CLAMPED ? MF_GATE_CLAMPED : EPI == 3 ? MF_ACT_GELU_TANH : MF_ACT_SILU;
+  return gated_product(g, u, act, ec);
+}
 
 // a sum on its way into a bfloat16 C: as it is (EPI 0) or through the activation EPI - 4 (EPI >= 4)
 template <int EPI> __device__ __forceinline__ float epi_value(unsigned bits) {
   const float v = __uint_as_float(bits);
-  return EPI >= 4 ? gate_act(v, EPI - 4) : v;
+  return EPI >= 4 && EPI < EPI_CLAMPED ? gate_act(v, EPI - 4) : v;
 }
 
 // Stores 32 consecutive columns of one row of the accumulator.
 template <int EPI>
-__device__ __forceinline__ void store_chunk(void* __restrict__ C, const unsigned (&r)[32], int row, int col, int N) {
-  if (EPI == 0 || EPI >= 4) {
+__device__ __forceinline__ void store_chunk(void* __restrict__ C, const unsigned (&r)[32], int row, int col, int N,
+                                            const EpiConst& ec) {
+  if (EPI == 0 || (EPI >= 4 && EPI < EPI_CLAMPED)) {
     __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(C) + (long long)row * N + col;
     if (col + 32 <= N && (((uintptr_t)dst) & 15) == 0) {
 #pragma unroll
@@ -126,7 +132,7 @@ __device__ __forceinline__ void store_chunk(void* __restrict__ C, const unsigned
       for (int j = 0; j < 32 && col + j < N; j++) dst[j] = __uint_as_float(r[j]);
     }
   } else {
-    // 32 columns = two groups of [8 gate | 8 up] -> 16 outputs at column col / 2 (EPI 2: SiLU, EPI 3: tanh-GELU)
+    // 32 columns = two groups of [8 gate | 8 up] -> 16 outputs at column col / 2 (EPI 2: SiLU, EPI 3: tanh-GELU, EPI_CLAMPED)
     __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(C) + (long long)row * (N / 2) + col / 2;
 #pragma unroll
     for (int grp = 0; grp < 2; grp++) {
@@ -134,7 +140,7 @@ __device__ __forceinline__ void store_chunk(void* __restrict__ C, const unsigned
       float o[8];
 #pragma unroll
       for (int j = 0; j < 8; j++)
-        o[j] = act_mul<EPI == 3 ? MF_ACT_GELU_TANH : MF_ACT_SILU>(__uint_as_float(r[grp * 16 + j]), __uint_as_float(r[grp * 16 + 8 + j]));
+        o[j] = epi_gate<EPI>(__uint_as_float(r[grp * 16 + j]), __uint_as_float(r[grp * 16 + 8 + j]), ec);
       if ((((uintptr_t)(dst + grp * 8)) & 15) == 0) {
         uint4 pk;
         pk.x = pack_bf16(o[0], o[1]); pk.y = pack_bf16(o[2], o[3]);
@@ -148,14 +154,14 @@ __device__ __forceinline__ void store_chunk(void* __restrict__ C, const unsigned
 }
 
 // EPI 0: C bfloat16 [M, N].  EPI 1: C float32 [M, N].  EPI 2: C bfloat16 [M, N/2] = silu(gate) * up.
-// EPI 4 + a: C bfloat16 [M, N] = act_a(A W^T), no gate (a: MF_ACT_*).
+// EPI 4 + a: C bfloat16 [M, N] = act_a(A W^T), no gate (a: MF_ACT_*).  EPI_CLAMPED: C bfloat16 [M, N/2], the clamped gate.
 // Persistent: a block walks tiles (tile, tile + grid, ...; the M index runs fastest, so blocks
 // that run together share tiles of W).  Two accumulators in tensor memory alternate, so the
 // epilogue of one tile runs while the products of the next are issued.
 template <int BN, int EPI>
 __global__ void __launch_bounds__(192)
 gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w, void* __restrict__ C,
-            int M, int N, int K, int* __restrict__ status) {
+            int M, int N, int K, EpiConst ec, int* __restrict__ status) {
   constexpr int B_BYTES = BN * BK * 2;
   constexpr int STAGE_BYTES = A_BYTES + B_BYTES;
   constexpr int TMEM_COLS = 2 * BN;
@@ -248,7 +254,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ C
         unsigned r[32];
         tmem_ld32(tmem_base + ((unsigned)(lg * 32) << 16) + acc * BN + (unsigned)(c * 32), r);
         const int col = n0 + c * 32;
-        if (row < M && col < N) store_chunk<EPI>(C, r, row, col, N);
+        if (row < M && col < N) store_chunk<EPI>(C, r, row, col, N, ec);
       }
       asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
       __syncwarp();
@@ -265,7 +271,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ C
 
 // ------------------------------------------------------------------ host side
 template <int BN, int EPI>
-int launch(const void* A, const void* W, void* C, int M, int N, int K, int* status, cudaStream_t stream) {
+int launch(const void* A, const void* W, void* C, int M, int N, int K, const EpiConst& ec, int* status, cudaStream_t stream) {
   CUtensorMap ma, mw;
   int rc = tma_host::bf16_map(A, M, K, BM, BK, &ma);
   if (rc) return rc;
@@ -283,8 +289,8 @@ int launch(const void* A, const void* W, void* C, int M, int N, int K, int* stat
   const int n_sms = mf_sm_count();
   if (n_sms <= 0) return MF_ERR_BAD_ARG;
   const int n_tiles = ((M + BM - 1) / BM) * ((N + BN - 1) / BN);
-  mf_count(EPI >= 4 ? MF_K_GEMM_TC_ACT : EPI >= 2 ? MF_K_GEMM_TC_SWIGLU : MF_K_GEMM_TC);
-  gemm_kernel<BN, EPI><<<n_tiles < n_sms ? n_tiles : n_sms, 192, smem, stream>>>(ma, mw, C, M, N, K, status);
+  mf_count(EPI >= 4 && EPI < EPI_CLAMPED ? MF_K_GEMM_TC_ACT : EPI >= 2 ? MF_K_GEMM_TC_SWIGLU : MF_K_GEMM_TC);
+  gemm_kernel<BN, EPI><<<n_tiles < n_sms ? n_tiles : n_sms, 192, smem, stream>>>(ma, mw, C, M, N, K, ec, status);
   return (int)cudaGetLastError();
 }
 
@@ -292,23 +298,27 @@ int launch(const void* A, const void* W, void* C, int M, int N, int K, int* stat
 
 // epilogue 0: C bfloat16 [M, N]; 1: C float32 [M, N]; 2 (SiLU), 3 (tanh-GELU): C bfloat16 [M, N/2] = act(gate) * up for a W
 // whose rows interleave gate and up in groups of 8 (N a multiple of 16); 4 + a: C bfloat16 [M, N] = act_a(A W^T) for the
-// activation a (MF_ACT_*), applied to the 32-bit sums.
+// activation a (MF_ACT_*), applied to the 32-bit sums; EPI_CLAMPED: as 2 and 3 with the clamped gate and its constants.
 // K must be a multiple of 8 and A, W 16-byte aligned (TMA strides).  `status` as in mf_stream_linear
 // (codes 11: producer, 12: MMA issuer, 13: epilogue).
-MF_API int mf_gemm_bf16(const void* A, const void* W, void* C, int M, int N, int K, int epilogue, int* status,
-                        cudaStream_t stream) {
+MF_API int mf_gemm_bf16(const void* A, const void* W, void* C, int M, int N, int K, int epilogue, float limit,
+                        float alpha, float up_off, int* status, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
-  if (K <= 0 || K % 8 || epilogue < 0 || epilogue >= 4 + MF_ACT_COUNT) return MF_ERR_BAD_ARG;
-  if ((epilogue == 2 || epilogue == 3) && N % 16) return MF_ERR_BAD_ARG;
+  if (K <= 0 || K % 8 || epilogue < 0 || epilogue > EPI_CLAMPED) return MF_ERR_BAD_ARG;
+  const EpiConst ec{limit, alpha, up_off, 0.f};
+  if ((epilogue == 2 || epilogue == 3 || epilogue == EPI_CLAMPED) && N % 16) return MF_ERR_BAD_ARG;
   if (((uintptr_t)A | (uintptr_t)W) & 15) return MF_ERR_BAD_ARG;
   const bool wide = N > 128;
   switch (epilogue) {
-    case 0: return wide ? launch<256, 0>(A, W, C, M, N, K, status, stream) : launch<128, 0>(A, W, C, M, N, K, status, stream);
-    case 1: return wide ? launch<256, 1>(A, W, C, M, N, K, status, stream) : launch<128, 1>(A, W, C, M, N, K, status, stream);
-    case 2: return wide ? launch<256, 2>(A, W, C, M, N, K, status, stream) : launch<128, 2>(A, W, C, M, N, K, status, stream);
-    case 3: return wide ? launch<256, 3>(A, W, C, M, N, K, status, stream) : launch<128, 3>(A, W, C, M, N, K, status, stream);
-    case 4: return wide ? launch<256, 4>(A, W, C, M, N, K, status, stream) : launch<128, 4>(A, W, C, M, N, K, status, stream);
-    case 5: return wide ? launch<256, 5>(A, W, C, M, N, K, status, stream) : launch<128, 5>(A, W, C, M, N, K, status, stream);
-    default: return wide ? launch<256, 6>(A, W, C, M, N, K, status, stream) : launch<128, 6>(A, W, C, M, N, K, status, stream);
+    case 0: return wide ? launch<256, 0>(A, W, C, M, N, K, ec, status, stream) : launch<128, 0>(A, W, C, M, N, K, ec, status, stream);
+    case 1: return wide ? launch<256, 1>(A, W, C, M, N, K, ec, status, stream) : launch<128, 1>(A, W, C, M, N, K, ec, status, stream);
+    case 2: return wide ? launch<256, 2>(A, W, C, M, N, K, ec, status, stream) : launch<128, 2>(A, W, C, M, N, K, ec, status, stream);
+    case 3: return wide ? launch<256, 3>(A, W, C, M, N, K, ec, status, stream) : launch<128, 3>(A, W, C, M, N, K, ec, status, stream);
+    case 4: return wide ? launch<256, 4>(A, W, C, M, N, K, ec, status, stream) : launch<128, 4>(A, W, C, M, N, K, ec, status, stream);
+    case 5: return wide ? launch<256, 5>(A, W, C, M, N, K, ec, status, stream) : launch<128, 5>(A, W, C, M, N, K, ec, status, stream);
+    case EPI_CLAMPED:
+      return wide ? launch<256, EPI_CLAMPED>(A, W, C, M, N, K, ec, status, stream)
+                  : launch<128, EPI_CLAMPED>(A, W, C, M, N, K, ec, status, stream);
+    default: return wide ? launch<256, 6>(A, W, C, M, N, K, ec, status, stream) : launch<128, 6>(A, W, C, M, N, K, ec, status, stream);
   }
 }

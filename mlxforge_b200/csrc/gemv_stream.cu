@@ -85,12 +85,16 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], unsigned a0, unsigned a1
 // 600 at 16384 x 2048; with the fence 0 of 600, whether the readers fence before they hand the stage
 // back or the producer fences once it has it: the latter is one thread's fence, off the readers' path).
 __device__ __forceinline__ void stage_is_mine() { asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory"); }
+// the gate of a product whose rows interleave gate and up (modes 1 to 3)
+__device__ __forceinline__ int gate_of_mode(int mode) {
+  return mode == 3 ? MF_GATE_CLAMPED : mode == 2 ? MF_ACT_GELU_TANH : MF_ACT_SILU;
+}
 __device__ __forceinline__ void consumer_sync() { asm volatile("bar.sync 1, %0;\n" ::"n"(CW * 32) : "memory"); }
 
 template <int NB, int ROWS, typename OutT>
 __global__ void __launch_bounds__((CW + 1) * 32)
 stream_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ W, OutT* __restrict__ out,
-              int M, int N, int K, int mode, int* __restrict__ status) {
+              int M, int N, int K, int mode, EpiConst ec, int* __restrict__ status) {
   constexpr int STAGES = Ring<ROWS>::STAGES;
   constexpr int STAGE_BYTES = ROWS * ROW_BYTES;
   extern __shared__ __align__(128) unsigned char smem[];
@@ -199,7 +203,8 @@ stream_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restri
         float sum = 0.f;
 #pragma unroll
         for (int w = 0; w < CW; w++) sum += red[(w * ROWS + r) * RED_M + m];
-        if (mode >= MF_STREAM_UNARY) sum = gate_act(sum, mode - MF_STREAM_UNARY);
+        if (mode == MF_STREAM_SOFTCAP) sum = soft_cap(sum, ec.cap);
+        else if (mode >= MF_STREAM_UNARY) sum = gate_act(sum, mode - MF_STREAM_UNARY);
         out[(long long)m * N + n0 + r] = from_f32<OutT>(sum);
       }
     } else {
@@ -213,7 +218,7 @@ stream_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restri
           gs += red[(w * ROWS + r) * RED_M + m];
           us += red[(w * ROWS + r + HALF) * RED_M + m];
         }
-        out[(long long)m * (N / 2) + tile * HALF + r] = from_f32<OutT>(gate_act(gs, mode == 2 ? MF_ACT_GELU_TANH : MF_ACT_SILU) * us);
+        out[(long long)m * (N / 2) + tile * HALF + r] = from_f32<OutT>(gated_product(gs, us, gate_of_mode(mode), ec));
       }
     }
     consumer_sync();       // `red` is free for the next tile
@@ -243,7 +248,7 @@ __device__ __forceinline__ void tma_load_3d(unsigned dst, const CUtensorMap* map
 template <int NB, int ROWS, int T_STAGES, typename OutT>
 __global__ void __launch_bounds__((CW + 1) * 32)
 stream_tmap_kernel(const __nv_bfloat16* __restrict__ x, const __grid_constant__ CUtensorMap map,
-                   OutT* __restrict__ out, int M, int N, int K, int mode, int* __restrict__ status) {
+                   OutT* __restrict__ out, int M, int N, int K, int mode, EpiConst ec, int* __restrict__ status) {
   constexpr int SUB = 16 / ROWS;                 // chunks of 64 per warp and stage (1 or 2)
   constexpr int KSTAGE = 512 * SUB;              // elements of K per stage
   constexpr int CHUNK_BYTES = ROWS * 128;
@@ -348,7 +353,8 @@ stream_tmap_kernel(const __nv_bfloat16* __restrict__ x, const __grid_constant__ 
         float sum = 0.f;
 #pragma unroll
         for (int w = 0; w < CW; w++) sum += red[(w * ROWS + r) * RED_M + m];
-        if (mode >= MF_STREAM_UNARY) sum = gate_act(sum, mode - MF_STREAM_UNARY);
+        if (mode == MF_STREAM_SOFTCAP) sum = soft_cap(sum, ec.cap);
+        else if (mode >= MF_STREAM_UNARY) sum = gate_act(sum, mode - MF_STREAM_UNARY);
         out[(long long)m * N + n0 + r] = from_f32<OutT>(sum);
       }
     } else {
@@ -362,7 +368,7 @@ stream_tmap_kernel(const __nv_bfloat16* __restrict__ x, const __grid_constant__ 
           gs += red[(w * ROWS + r) * RED_M + m];
           us += red[(w * ROWS + r + HALF) * RED_M + m];
         }
-        out[(long long)m * (N / 2) + tile * HALF + r] = from_f32<OutT>(gate_act(gs, mode == 2 ? MF_ACT_GELU_TANH : MF_ACT_SILU) * us);
+        out[(long long)m * (N / 2) + tile * HALF + r] = from_f32<OutT>(gated_product(gs, us, gate_of_mode(mode), ec));
       }
     }
     consumer_sync();       // `red` is free for the next tile
@@ -370,8 +376,8 @@ stream_tmap_kernel(const __nv_bfloat16* __restrict__ x, const __grid_constant__ 
 }
 
 template <int NB, int ROWS, int T_STAGES, typename OutT>
-int launch_tmap(const __nv_bfloat16* x, const __nv_bfloat16* W, OutT* out, int M, int N, int K, int mode, int* status,
-                int n_sms, cudaStream_t stream) {
+int launch_tmap(const __nv_bfloat16* x, const __nv_bfloat16* W, OutT* out, int M, int N, int K, int mode,
+                const EpiConst& ec, int* status, int n_sms, cudaStream_t stream) {
   const size_t smem = 1024 + (size_t)T_STAGES * T_STAGE_BYTES + 2 * T_STAGES * 8 + (size_t)CW * ROWS * (NB * 8 + 1) * 4;
   static DeviceOnce once;
   const int dev_ = mf_current_device();
@@ -392,12 +398,12 @@ int launch_tmap(const __nv_bfloat16* x, const __nv_bfloat16* W, OutT* out, int M
   const int grid = (n_tiles + rounds - 1) / rounds;
   mf_count(MF_K_STREAM_TMAP);
   return (int)launch_dep(stream_tmap_kernel<NB, ROWS, T_STAGES, OutT>, dim3(grid), dim3((CW + 1) * 32), smem, stream, x, map,
-                         out, M, N, K, mode, status);
+                         out, M, N, K, mode, ec, status);
 }
 
 template <int NB, int ROWS, typename OutT>
-int launch_one(const __nv_bfloat16* x, const __nv_bfloat16* W, OutT* out, int M, int N, int K, int mode, int* status,
-               int n_sms, cudaStream_t stream) {
+int launch_one(const __nv_bfloat16* x, const __nv_bfloat16* W, OutT* out, int M, int N, int K, int mode,
+                const EpiConst& ec, int* status, int n_sms, cudaStream_t stream) {
   constexpr int STAGES = Ring<ROWS>::STAGES;
   const size_t smem = (size_t)STAGES * ROWS * ROW_BYTES + 2 * STAGES * 8 + (size_t)CW * ROWS * (NB * 8 + 1) * 4;
   static DeviceOnce once;
@@ -414,12 +420,12 @@ int launch_one(const __nv_bfloat16* x, const __nv_bfloat16* W, OutT* out, int M,
   const int grid = n_tiles < 2 * n_sms ? n_tiles : 2 * n_sms;
   mf_count(MF_K_STREAM_ROWS);
   return (int)launch_dep(stream_kernel<NB, ROWS, OutT>, dim3(grid), dim3((CW + 1) * 32), smem, stream, x, W, out, M,
-                         N, K, mode, status);
+                         N, K, mode, ec, status);
 }
 
 template <typename OutT>
-int dispatch(const __nv_bfloat16* x, const __nv_bfloat16* W, OutT* out, int M, int N, int K, int mode, int* status,
-             cudaStream_t stream) {
+int dispatch(const __nv_bfloat16* x, const __nv_bfloat16* W, OutT* out, int M, int N, int K, int mode,
+                const EpiConst& ec, int* status, cudaStream_t stream) {
   const int n_sms = mf_sm_count();
   if (n_sms <= 0) return MF_ERR_BAD_ARG;
   // few output rows: tiles of 8 rows, so that there are blocks for every SM
@@ -433,20 +439,20 @@ int dispatch(const __nv_bfloat16* x, const __nv_bfloat16* W, OutT* out, int M, i
     // has to keep nearly all of its shared memory on the way (four stages: 1.141 ms for a decode step
     // of batch 8, six: 1.133, and 1.102 against 1.117 once the kernels before let this one start early).
     if (M <= 8)
-      return small ? launch_tmap<1, 8, 6, OutT>(x, W, out, M, N, K, mode, status, n_sms, stream)
-                   : launch_tmap<1, 16, 6, OutT>(x, W, out, M, N, K, mode, status, n_sms, stream);
+      return small ? launch_tmap<1, 8, 6, OutT>(x, W, out, M, N, K, mode, ec, status, n_sms, stream)
+                   : launch_tmap<1, 16, 6, OutT>(x, W, out, M, N, K, mode, ec, status, n_sms, stream);
     if (M <= 16)
-      return small ? launch_tmap<2, 8, 6, OutT>(x, W, out, M, N, K, mode, status, n_sms, stream)
-                   : launch_tmap<2, 16, 6, OutT>(x, W, out, M, N, K, mode, status, n_sms, stream);
+      return small ? launch_tmap<2, 8, 6, OutT>(x, W, out, M, N, K, mode, ec, status, n_sms, stream)
+                   : launch_tmap<2, 16, 6, OutT>(x, W, out, M, N, K, mode, ec, status, n_sms, stream);
     return MF_ERR_BAD_ARG;
   }
   if (M <= 8) {
-    return small ? launch_one<1, 8, OutT>(x, W, out, M, N, K, mode, status, n_sms, stream)
-                 : launch_one<1, 16, OutT>(x, W, out, M, N, K, mode, status, n_sms, stream);
+    return small ? launch_one<1, 8, OutT>(x, W, out, M, N, K, mode, ec, status, n_sms, stream)
+                 : launch_one<1, 16, OutT>(x, W, out, M, N, K, mode, ec, status, n_sms, stream);
   }
   if (M <= 16) {
-    return small ? launch_one<2, 8, OutT>(x, W, out, M, N, K, mode, status, n_sms, stream)
-                 : launch_one<2, 16, OutT>(x, W, out, M, N, K, mode, status, n_sms, stream);
+    return small ? launch_one<2, 8, OutT>(x, W, out, M, N, K, mode, ec, status, n_sms, stream)
+                 : launch_one<2, 16, OutT>(x, W, out, M, N, K, mode, ec, status, n_sms, stream);
   }
   return MF_ERR_BAD_ARG;
 }
@@ -462,20 +468,22 @@ MF_API int mf_set_stream_tensor_copies(int on) {
   return 0;
 }
 
-// mode 0: out [M, N] in out_dtype.  mode 1 (SiLU) and 2 (tanh form of GELU): W rows interleave gate and up in groups of 8 (N a
+// mode 0: out [M, N] in out_dtype.  mode 1 (SiLU), 2 (tanh form of GELU) and 3 (the clamped gate with its three constants): W rows interleave gate and up in groups of 8 (N a
 // multiple of 16) and out is [M, N / 2] = act(gate) * up.  mode MF_STREAM_UNARY + a: out [M, N] = act_a(x W^T), the
-// activation (MF_ACT_*) applied to the 32-bit sums before they are rounded.  K must be a multiple of 8 and x, W
+// activation (MF_ACT_*) applied to the 32-bit sums before they are rounded; MF_STREAM_SOFTCAP: cap tanh(sum / cap).  K must be a multiple of 8 and x, W
 // 16-byte aligned.  `status`: a device int (may be null) that receives a non-zero code if a wait
 // inside the kernel ran out (1: producer, 2: consumer).
 MF_API int mf_stream_linear(const void* x, const void* W, void* out, int out_dtype, int M, int N, int K, int mode,
-                            int* status, cudaStream_t stream) {
+                            float limit, float alpha, float up_off, float cap, int* status, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
-  const bool unary = mode >= MF_STREAM_UNARY && mode < MF_STREAM_UNARY + MF_ACT_COUNT;
-  if (K <= 0 || K % 8 || M > 16 || mode < 0 || (mode > 2 && !unary)) return MF_ERR_BAD_ARG;
+  const bool unary = (mode >= MF_STREAM_UNARY && mode < MF_STREAM_UNARY + MF_ACT_COUNT) || mode == MF_STREAM_SOFTCAP;
+  if (K <= 0 || K % 8 || M > 16 || mode < 0 || (mode > 3 && !unary)) return MF_ERR_BAD_ARG;
+  if (mode == MF_STREAM_SOFTCAP && !(cap > 0.f)) return MF_ERR_BAD_ARG;
+  const EpiConst ec{limit, alpha, up_off, cap};
   if (mode != 0 && !unary && N % 16) return MF_ERR_BAD_ARG;
   if (((uintptr_t)x | (uintptr_t)W) & 15) return MF_ERR_BAD_ARG;
   const __nv_bfloat16 *xx = (const __nv_bfloat16*)x, *ww = (const __nv_bfloat16*)W;
-  if (out_dtype == MF_BF16) return dispatch<__nv_bfloat16>(xx, ww, (__nv_bfloat16*)out, M, N, K, mode, status, stream);
-  if (out_dtype == MF_F32) return dispatch<float>(xx, ww, (float*)out, M, N, K, mode, status, stream);
+  if (out_dtype == MF_BF16) return dispatch<__nv_bfloat16>(xx, ww, (__nv_bfloat16*)out, M, N, K, mode, ec, status, stream);
+  if (out_dtype == MF_F32) return dispatch<float>(xx, ww, (float*)out, M, N, K, mode, ec, status, stream);
   return MF_ERR_BAD_DTYPE;
 }

@@ -17,7 +17,8 @@ const char* const kNames[MF_K_COUNT] = {
     "unary_act",        "gemm_tc_act",      "conv_input",       "postnorm_add",     "qk_norm_rope",
     "rotate_rows",      "gdelta_prepare",   "gdelta_recurrence",
     "conv_act",         "decay_recurrence", "decay_local",      "scan_combine",     "gated_norm",
-    "selective_scan",   "scan_local",       "low_rank",
+    "selective_scan",   "scan_local",       "low_rank",         "post_norm",      "qkv_conv",
+    "soft_cap",
 };
 int g_sm_count[MF_MAX_DEVICES] = {};
 }  // namespace

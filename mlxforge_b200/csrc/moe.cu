@@ -1,6 +1,7 @@
 // Mixture of experts: the router's choice and the experts' feed-forward.
 //
-// Router (32-bit): s = sigmoid(z) over E experts, or s = softmax(z) over them (`mode`).  The
+// Router (32-bit): s = sigmoid(z) over E experts, or s = softmax(z) over them (`mode`), z with
+// `logit_bias` added where there is one.  The
 // experts form `n_groups` equal groups of neighbours; a group's score is the sum of its two
 // largest s, and only experts of the `keep` best groups can be chosen (n_groups = 0: no such
 // limit).  The `top` allowed experts with the largest s + bias (`bias`: one number per expert
@@ -28,7 +29,7 @@ __device__ __forceinline__ float moe_sigmoid(float x) { return 1.0f / (1.0f + ex
 // one warp per token; dynamic shared memory per warp: s[E], sel[E], gs[n_groups]
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ z, int ldz, int E, int n_groups, int keep, int top, float route_scale,
-                 int mode, const float* __restrict__ bias, int* __restrict__ ids, float* __restrict__ weights, int T) {
+                 int mode, const float* __restrict__ logit_bias, const float* __restrict__ bias, int* __restrict__ ids, float* __restrict__ weights, int T) {
   extern __shared__ float sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * (blockDim.x >> 5) + warp;
@@ -41,17 +42,20 @@ moe_route_kernel(const float* __restrict__ z, int ldz, int E, int n_groups, int 
   const bool renorm = (mode & 2) != 0;       // the chosen weights divided by their sum (+ 1e-20)
   if (mode & 1) {
     float m = -INFINITY;
-    for (int e = lane; e < E; e += 32) m = fmaxf(m, zr[e]);
+    for (int e = lane; e < E; e += 32) {
+      s[e] = logit_bias ? zr[e] + logit_bias[e] : zr[e];
+      m = fmaxf(m, s[e]);
+    }
     m = warp_max(m);
     float sum = 0.f;
     for (int e = lane; e < E; e += 32) {
-      s[e] = expf(zr[e] - m);
+      s[e] = expf(s[e] - m);
       sum += s[e];
     }
     sum = warp_sum(sum);
     for (int e = lane; e < E; e += 32) s[e] = s[e] / sum;
   } else {
-    for (int e = lane; e < E; e += 32) s[e] = moe_sigmoid(zr[e]);
+    for (int e = lane; e < E; e += 32) s[e] = moe_sigmoid(logit_bias ? zr[e] + logit_bias[e] : zr[e]);
   }
   for (int e = lane; e < E; e += 32) sel[e] = bias ? s[e] + bias[e] : s[e];
   __syncwarp();
@@ -117,7 +121,8 @@ moe_route_kernel(const float* __restrict__ z, int ldz, int E, int n_groups, int 
 }
 
 MF_API int mf_moe_route(const float* z, int ldz, int T, int E, int n_groups, int keep, int top, float route_scale,
-                        int mode, const float* bias, int* ids, float* weights, cudaStream_t stream) {
+                        int mode, const float* logit_bias, const float* bias, int* ids, float* weights,
+                        cudaStream_t stream) {
   if (T <= 0) return 0;
   if (E <= 0 || top <= 0 || top > E || ldz < E || mode < 0 || mode > 3) return MF_ERR_BAD_ARG;
   if (n_groups > 0 && (E % n_groups || keep < 1 || keep > n_groups || (long long)keep * (E / n_groups) < top))
@@ -126,8 +131,8 @@ MF_API int mf_moe_route(const float* z, int ldz, int T, int E, int n_groups, int
   const size_t smem = (size_t)4 * per_warp * sizeof(float);
   if (smem > 48 * 1024) return MF_ERR_BAD_ARG;
   mf_count(MF_K_MOE_ROUTE);
-  moe_route_kernel<<<(T + 3) / 4, 128, smem, stream>>>(z, ldz, E, n_groups, keep, top, route_scale, mode, bias, ids,
-                                                       weights, T);
+  moe_route_kernel<<<(T + 3) / 4, 128, smem, stream>>>(z, ldz, E, n_groups, keep, top, route_scale, mode,
+                                                       logit_bias, bias, ids,                                                       weights, T);
   return (int)cudaGetLastError();
 }
 

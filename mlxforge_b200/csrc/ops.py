@@ -7,7 +7,7 @@ from __future__ import annotations
 
 from ctypes import c_void_p
 from functools import lru_cache
-from typing import Optional
+from typing import NamedTuple, Optional
 
 import torch
 
@@ -64,6 +64,30 @@ def add_rmsnorm(resid: torch.Tensor, delta: Optional[torch.Tensor], weight: torc
                                    _stream()), "add_rmsnorm")
 
 
+NORM_KINDS = {None: 0, "rms": 1, "layer": 2}
+
+
+def post_norm(resid: torch.Tensor, y: Optional[torch.Tensor], y_weight: Optional[torch.Tensor], y_kind: Optional[str],
+              y_eps: float, weight: torch.Tensor, kind: str, eps: float, out: torch.Tensor,
+              rows: Optional[torch.Tensor] = None) -> None:
+    """``resid += norm(y) * y_weight`` (``y_kind`` None: ``resid += y``; ``y`` None: nothing), then
+    ``out = norm(resid) * weight``; each norm ``"rms"`` or ``"layer"`` (mean taken off, no bias).  With ``rows``
+    only those rows are produced and ``resid`` stays."""
+    _need_cuda(resid, y, y_weight, weight, out, rows)
+    check(library().mf_post_norm(resid.data_ptr(), _ptr(y), dtype_code(y) if y is not None else dtype_code(out),
+                                 _ptr(y_weight), NORM_KINDS[y_kind], y_eps, weight.data_ptr(), NORM_KINDS[kind], eps,
+                                 out.data_ptr(), dtype_code(out), _ptr(rows), out.shape[0], resid.shape[-1], _stream()),
+          "post_norm")
+
+
+def soft_cap(x: torch.Tensor, cap: float) -> None:
+    """``x = cap tanh(x / cap)`` in place (32-bit)."""
+    _need_cuda(x)
+    if x.dtype != torch.float32:
+        raise KernelError("soft_cap: 32-bit values")
+    check(library().mf_soft_cap(x.data_ptr(), x.numel(), float(cap), _stream()), "soft_cap")
+
+
 def residual_add(resid: torch.Tensor, delta: torch.Tensor) -> None:
     _need_cuda(resid, delta)
     check(library().mf_residual_add(resid.data_ptr(), delta.data_ptr(), dtype_code(delta), resid.numel(),
@@ -85,6 +109,26 @@ def rope_kv_write(qkv: torch.Tensor, positions: torch.Tensor, seq_of_token: torc
 
 ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu2": 2}
 STREAM_UNARY = 16      # mode of the few-row product with an activation without a gate: STREAM_UNARY + code
+STREAM_SOFTCAP = 32    # mode of the few-row product whose sums pass a soft cap
+
+
+class ClampedGate(NamedTuple):
+    """A gate beside the names above: ``min(g, limit)`` and ``clamp(u, -limit, limit)``, then
+    ``g sigmoid(alpha g) (u + up_offset)``.  Taken wherever gate and up are multiplied."""
+
+    limit: float
+    alpha: float = 1.702
+    up_offset: float = 1.0
+
+
+GATE_CLAMPED = 8
+
+
+def gate_code(act):
+    """(code, limit, alpha, up_offset) of a gate: an activation's name or a ``ClampedGate``."""
+    if isinstance(act, ClampedGate):
+        return GATE_CLAMPED, act.limit, act.alpha, act.up_offset
+    return activation_code(act), 0.0, 1.0, 0.0
 
 
 def activation_code(act: str) -> int:
@@ -94,11 +138,11 @@ def activation_code(act: str) -> int:
         raise KernelError(f"unknown gate activation '{act}' (one of {sorted(ACTIVATIONS)})") from None
 
 
-def swiglu(gu: torch.Tensor, out: torch.Tensor, group: int, act: str = "silu") -> None:
-    """out = act(gate) * up for gate and up interleaved in groups of ``group`` columns."""
+def swiglu(gu: torch.Tensor, out: torch.Tensor, group: int, act="silu") -> None:
+    """out = act(gate) * up (or a ``ClampedGate``) for gate and up interleaved in groups of ``group`` columns."""
     _need_cuda(gu, out)
     T, I = out.shape
-    check(library().mf_gated_act(gu.data_ptr(), out.data_ptr(), dtype_code(gu), T, I, group, activation_code(act),
+    check(library().mf_gated_act(gu.data_ptr(), out.data_ptr(), dtype_code(gu), T, I, group, *gate_code(act),
                                  _stream()), "gated_act")
 
 
@@ -431,11 +475,12 @@ def set_stream_tensor_copies(on: bool) -> None:
 
 
 def stream_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: bool = False,
-                  act: str = "silu", unary: bool = False) -> None:
+                  act="silu", unary: bool = False, softcap: float = 0.0) -> None:
     """out = x @ w^T for at most ``stream_max_rows()`` rows of bfloat16 x (out bfloat16 or
     float32), the weights streamed by bulk copies (see gemv_stream.cu); with ``swiglu`` the rows
     of w interleave gate and up in groups of 8 and out [M, N/2] is act(gate) * up; with ``unary``
-    out [M, N] is act(x @ w^T), the activation applied to the 32-bit sums.
+    out [M, N] is act(x @ w^T), the activation applied to the 32-bit sums; with ``softcap``
+    out is ``softcap * tanh(x @ w^T / softcap)``.
     The kernel starts fetching ``w`` before it waits for the kernel launched before it, so
     ``w`` must not be the output of that kernel (the engine's weights are written once, at
     load time)."""
@@ -447,10 +492,16 @@ def stream_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: b
         raise KernelError(f"stream_linear: shapes {tuple(x.shape)} x {tuple(w.shape)}^T -> {tuple(out.shape)}")
     if swiglu and unary:
         raise KernelError("stream_linear: an activation with a gate or without one, not both")
-    mode = 1 + activation_code(act) if swiglu else (STREAM_UNARY + activation_code(act) if unary else 0)
+    if softcap and (swiglu or unary):
+        raise KernelError("stream_linear: a soft cap or an activation, not both")
+    code, limit, alpha, up_off = gate_code(act)
+    mode = (3 if code == GATE_CLAMPED else 1 + code) if swiglu else STREAM_UNARY + activation_code(act) if unary else \
+        STREAM_SOFTCAP if softcap else 0
+    if swiglu and act == "relu2":
+        raise KernelError("stream_linear: the gated epilogue has SiLU, the tanh form of GELU and the clamped gate")
     check(library().mf_stream_linear(x.data_ptr(), w.data_ptr(), out.data_ptr(), dtype_code(out), M, N, K,
-                                     mode, kernel_status(x.device).data_ptr(), _stream()),
-          "stream_linear")
+                                     mode, limit, alpha, up_off, float(softcap), kernel_status(x.device).data_ptr(),
+                                     _stream()), "stream_linear")
 
 
 def mid_rows_range():
@@ -488,7 +539,7 @@ def gemm_ok(x: torch.Tensor, w: torch.Tensor) -> bool:
             and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
-def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: bool = False, act: str = "silu",
+def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: bool = False, act="silu",
               unary: bool = False) -> None:
     """out = x @ w^T on the tcgen05 tensor cores (bfloat16 operands; out bfloat16 or float32);
     with ``swiglu`` the rows of w interleave gate and up in groups of 8 and out is
@@ -506,9 +557,10 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, swiglu: bool 
         raise KernelError("gemm_bf16: an activation with a gate or without one, not both")
     if swiglu and act == "relu2":
         raise KernelError("gemm_bf16: the gated epilogue has SiLU and the tanh form of GELU")
-    epi = (2 + activation_code(act) if swiglu else 4 + activation_code(act) if unary
+    code, limit, alpha, up_off = gate_code(act)
+    epi = ((4 + len(ACTIVATIONS) if code == GATE_CLAMPED else 2 + code) if swiglu else 4 + activation_code(act) if unary
            else (1 if out.dtype == torch.float32 else 0))
-    check(library().mf_gemm_bf16(x.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, epi,
+    check(library().mf_gemm_bf16(x.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, epi, limit, alpha, up_off,
                                  kernel_status(x.device).data_ptr(), _stream()), "gemm_bf16")
 
 
@@ -817,6 +869,34 @@ def qk_norm_rope(proj: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, v_d
                                     v_pool.data_ptr(), int(write_kv), _stream()), "qk_norm_rope")
 
 
+def qkv_conv_ok(head_dim: int, v_dim: int, taps: int, ld: int, rot: int) -> bool:
+    """Whether ``qkv_conv`` takes these sizes."""
+    return bool(library().mf_qkv_conv_ok(head_dim, v_dim, taps, ld, rot))
+
+
+def qkv_conv(proj: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, v_dim: int, rot: int, eps: float,
+             conv_w: torch.Tensor, q_w, k_w, inv_f, inv_d, state: Optional[torch.Tensor], batch,
+             block_table: torch.Tensor, page_size: int, q_out: torch.Tensor, k_pool: torch.Tensor,
+             v_pool: torch.Tensor) -> None:
+    """From 32-bit projections [queries | keys | values] (``n_kv`` 0: queries alone): the causal convolution
+    over time (``conv_w`` [channels, taps], the last taps-1 rows of every sequence at the start of its slot of
+    ``state``, which move on), the norms per head (``q_w``, ``k_w`` [head_dim]; None: no norm), the rotation of
+    half-split pairs, and the cache write."""
+    _need_cuda(proj, conv_w, q_w, k_w, inv_f, inv_d, state, block_table, q_out, k_pool, v_pool)
+    T, taps = proj.shape[0], conv_w.shape[1]
+    if proj.dtype != torch.float32 or conv_w.shape[0] != n_heads * head_dim + n_kv * (head_dim + v_dim):
+        raise KernelError("qkv_conv: 32-bit projections and a row of taps per channel")
+    if taps > 1 and (state is None or state.dtype != torch.float32):
+        raise KernelError("qkv_conv: a convolution of several taps needs a state")
+    check(library().mf_qkv_conv(proj.data_ptr(), proj.shape[1], dtype_code(q_out), T, n_heads, n_kv, head_dim, v_dim, rot,
+                                eps, conv_w.data_ptr(), taps, _ptr(q_w), _ptr(k_w), _ptr(inv_f), _ptr(inv_d), _ptr(state),
+                                state.stride(0) if state is not None else 0, 0, batch.positions.data_ptr(),
+                                batch.seq_of_token.data_ptr(), batch.seq_q_start.data_ptr(), batch.seq_q_len.data_ptr(),
+                                batch.slots.data_ptr(), batch.n_seqs, block_table.data_ptr(), block_table.shape[1],
+                                page_size, q_out.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), _stream()), "qkv_conv",
+          launches=2 if taps > 1 and T != batch.n_seqs else 1)
+
+
 def rotate_rows(x: torch.Tensor, n_heads: int, d: int, rot: int, positions: torch.Tensor, inv_f, inv_d,
                 sign: float) -> None:
     """The heads of every row of ``x`` [T, n_heads * d] turned in place by ``sign * position`` (half-split pairs
@@ -983,14 +1063,15 @@ def low_rank(low: torch.Tensor, ld: int, wt: torch.Tensor, bias: Optional[torch.
 
 def moe_route(z: torch.Tensor, n_groups: int, keep: int, top: int, route_scale: float, ids: torch.Tensor,
               weights: torch.Tensor, n_experts: Optional[int] = None, softmax: bool = False,
-              bias: Optional[torch.Tensor] = None, renormalize: bool = False) -> None:
+              bias: Optional[torch.Tensor] = None, renormalize: bool = False,
+              logit_bias: Optional[torch.Tensor] = None) -> None:
     """The router's choice from logits ``z`` [T, >= n_experts] (the first ``n_experts`` columns of every row;
     default all): scores by sigmoid or, with ``softmax``, by a softmax over the experts; ``bias`` (32-bit, one
-    per expert) is added for the choice only; ``renormalize``: the chosen weights are divided by their sum."""
-    _need_cuda(z, ids, weights, bias)
+    per expert) is added for the choice only; ``logit_bias`` (likewise) is added to the logits; ``renormalize``: the chosen weights are divided by their sum."""
+    _need_cuda(z, ids, weights, bias, logit_bias)
     E = z.shape[1] if n_experts is None else n_experts
     check(library().mf_moe_route(z.data_ptr(), z.shape[1], z.shape[0], E, n_groups, keep, top, route_scale,
-                                 (1 if softmax else 0) | (2 if renormalize else 0), _ptr(bias), ids.data_ptr(),
+                                 (1 if softmax else 0) | (2 if renormalize else 0), _ptr(logit_bias), _ptr(bias), ids.data_ptr(),
                                  weights.data_ptr(), _stream()),
           "moe_route")
 

@@ -130,6 +130,16 @@ class Runtime:
         return ((self.mid_rows_enabled or self.gemm_backend == "tcgen05") and self.gemm_backend != "library"
                 and x.shape[0] <= self.mid_max_rows and ops.gemm_ok(x, w))
 
+    def linear_softcap(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, cap: float) -> torch.Tensor:
+        """``out = cap tanh(x w^T / cap)`` in 32-bit: in the epilogue of the few-row product, else in place
+        behind the product."""
+        if x.dtype == torch.bfloat16 and self._skinny(x, w):
+            ops.stream_linear(x, w, out, softcap=cap)
+            return out
+        self.linear(x, w, out)
+        ops.soft_cap(out, cap)
+        return out
+
     def linear_act(self, x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, act: str) -> torch.Tensor:
         """``out = act(x w^T)`` for an activation without a gate (``ops.ACTIVATIONS``), applied to the 32-bit
         sums where the product's kernel has it in its epilogue (the few-row kernel and the tcgen05 one),
@@ -148,9 +158,9 @@ class Runtime:
         return out
 
     def linear_swiglu(self, x: torch.Tensor, w_gu: torch.Tensor, group: int, out: torch.Tensor,
-                      act: str = "silu") -> torch.Tensor:
+                      act="silu") -> torch.Tensor:
         """``out = act(x Wg^T) * (x Wu^T)`` for a matrix whose rows interleave gate and
-        up in groups of ``group``; ``act`` is ``"silu"`` or ``"gelu_tanh"``.  Few bfloat16 rows: one
+        up in groups of ``group``; ``act`` is ``"silu"``, ``"gelu_tanh"`` or an ``ops.ClampedGate``.  Few bfloat16 rows: one
         kernel with the product in its epilogue; otherwise the product, then the elementwise kernel."""
         if group == 8 and w_gu.shape[0] % 16 == 0 and self._skinny(x, w_gu):
             ops.stream_linear(x, w_gu, out, swiglu=True, act=act)

@@ -5,13 +5,14 @@ head) with the head applied only to the rows whose logits were asked for.
 """
 from __future__ import annotations
 
+from dataclasses import replace
 from typing import Dict, List, Optional
 
 import torch
 
 from ..cache.manager import CacheLayout, GroupLayout
-from ..parts.base import (EMBEDDINGS, HEADS, NORMS, FixedState, ModelSpec, PagedKV, TensorSpec, build_layer,
-                          build_part)
+from ..parts.base import (EMBEDDINGS, HEADS, NORMS, FixedState, ModelSpec, PagedKV, TensorSpec, build_layer, build_part,
+                          flatten_needs)
 from ..weights.loader import WeightError, load_tensors
 
 
@@ -80,6 +81,31 @@ class DecoderModel:
         return total
 
     # ------------------------------------------------------------------ cache
+    def _needs(self) -> List[tuple]:
+        """What every item of the schedule keeps per request, as a flat tuple.  Items that read another's cache
+        may see further back than it does: the owner's pages are then kept for the widest of them."""
+        needs = [flatten_needs(self.blocks[item.layer].cache_need()) for item in self.spec.schedule]
+        for i, item in enumerate(self.spec.schedule):
+            if item.cache_of is None:
+                continue
+            root = item.cache_of
+            while self.spec.schedule[root].cache_of is not None:
+                root = self.spec.schedule[root].cache_of
+            own = [n for n in needs[i] if isinstance(n, PagedKV)]
+            src = [k for k, n in enumerate(needs[root]) if isinstance(n, PagedKV)]
+            if len(src) != 1:
+                raise ValueError(f"schedule item {i} reads the cache of item {item.cache_of}, which has none to share")
+            need = needs[root][src[0]]
+            if len(own) != 1 or (own[0].n_kv_heads, own[0].head_dim, own[0].value_dim, own[0].values_in_keys) != (
+                    need.n_kv_heads, need.head_dim, need.value_dim, need.values_in_keys):
+                raise ValueError(f"schedule item {i} cannot read a cache of another geometry")
+            window = 0 if 0 in (own[0].window, need.window) else max(own[0].window, need.window)
+            widened = list(needs[root])
+            widened[src[0]] = replace(need, window=window, chunk=need.chunk if own[0].chunk == need.chunk else 0,
+                                      keep_first=max(own[0].keep_first, need.keep_first))
+            needs[root] = tuple(widened)
+        return needs
+
     def _layout(self) -> CacheLayout:
         paged: List[list] = []     # [need, lanes]
         state: List[list] = []
@@ -100,26 +126,19 @@ class DecoderModel:
             groups.append([need, 1])
             return (kind, len(groups) - 1, 0)
 
-        for i, item in enumerate(self.spec.schedule):
-            if item.cache_of is not None:
-                src = item_lane[item.cache_of]
-                need = self.blocks[item.layer].cache_need()
-                if src is None or isinstance(src[0], tuple) or src[0] != "paged":
-                    raise ValueError(f"schedule item {i} reads the cache of item {item.cache_of}, which has none to share")
-                src_need = paged[src[1]][0]
-                if not isinstance(need, PagedKV) or (need.n_kv_heads, need.head_dim, need.value_dim) != (
-                        src_need.n_kv_heads, src_need.head_dim, src_need.value_dim):
-                    raise ValueError(f"schedule item {i} cannot read a cache of another geometry")
-                item_lane.append(src)
-                continue
-            need = self.blocks[item.layer].cache_need()
-            if isinstance(need, tuple):
-                # several needs: the item's lanes are a tuple in the order of the needs
-                item_lane.append(tuple(place(n, item.layer) for n in need))
-            else:
-                item_lane.append(None if need is None else place(need, item.layer))
+        for i, (item, needs) in enumerate(zip(self.spec.schedule, self._needs())):
+            # an item that reads another's cache has the owner's pages in place of its own, and its own state
+            lanes = tuple(self._paged_lane(item_lane[item.cache_of])
+                          if item.cache_of is not None and isinstance(n, PagedKV) else place(n, item.layer) for n in needs)
+            # several needs: the item's lanes are a tuple in the order of the needs
+            item_lane.append(None if not lanes else lanes[0] if len(lanes) == 1 else lanes)
         return CacheLayout(tuple(GroupLayout(n, l) for n, l in paged), tuple(GroupLayout(n, l) for n, l in state),
                            tuple(item_lane))
+
+    @staticmethod
+    def _paged_lane(where) -> tuple:
+        """The lane of pages among an item's lanes."""
+        return next(w for w in (where if isinstance(where[0], tuple) else (where,)) if w[0] == "paged")
 
     # ------------------------------------------------------------------ forward
     def forward(self, batch, cache) -> Optional[torch.Tensor]:

@@ -16,7 +16,7 @@ from typing import Dict
 import torch
 
 from ..csrc import ops
-from .base import POSITIONS, Mixer, PagedKV, PartSpec, TensorSpec, build_part, register_mixer
+from .base import POSITIONS, FixedState, Mixer, PagedKV, PartSpec, TensorSpec, build_part, register_mixer
 
 
 def paged_attention(rt, batch, q, lane, out, n_heads: int, scale: float, window: int) -> None:
@@ -122,9 +122,10 @@ class AttentionMixer(Mixer):
 
 
 def options_paged_attention(rt, batch, q, lane, out, n_heads: int, scale: float, window: int = 0, keep_first: int = 0,
-                            sink=None, gate=None, gate_ld: int = 0) -> None:
+                            sink=None, gate=None, gate_ld: int = 0, softcap: float = 0.0) -> None:
     """Attention over ``lane`` with the options beyond a window: values of their own width or inside the
-    keys (the lane's need says which), kept first keys, a sink, a gate on the output.  bfloat16 with sizes
+    keys (the lane's need says which), kept first keys, a sink, a gate on the output, a soft cap on the scaled
+    scores.  bfloat16 with sizes
     the tensor-core kernels take: the sequences that bring one token (the batch lays them out first) go to
     the split-key decode kernel, portions of prompts to the prefill kernel; the 32-bit path and other sizes
     take the block-per-token kernel."""
@@ -134,7 +135,7 @@ def options_paged_attention(rt, batch, q, lane, out, n_heads: int, scale: float,
     if q.dtype != torch.bfloat16 or not ops.attention_tc_ok(need.head_dim, vd, lane.page_size):
         ops.attention_generic_ex(q, lane.k, lane.v, out, batch.positions, batch.seq_of_token, table, lane.page_size,
                                  n_heads, need.n_kv_heads, need.head_dim, scale, window, vd,
-                                 need.head_dim if in_k else vd, keep_first, sink, gate, gate_ld)
+                                 need.head_dim if in_k else vd, keep_first, sink, gate, gate_ld, softcap)
         return
     nd = batch.n_decode
     if nd > 0:
@@ -142,12 +143,13 @@ def options_paged_attention(rt, batch, q, lane, out, n_heads: int, scale: float,
         ops.attention_decode_ex(q[:nd], lane.k, lane.v, out[:nd], rt.buffer("attn.part_o", (n_o,), torch.float32),
                                 rt.buffer("attn.part_ml", (n_ml,), torch.float32), batch.positions[:nd],
                                 batch.seq_of_token[:nd], table, lane.page_size, n_heads, need.n_kv_heads,
-                                need.head_dim, scale, window, batch.max_ctx, vd, in_k, keep_first, sink, gate, gate_ld)
+                                need.head_dim, scale, window, batch.max_ctx, vd, in_k, keep_first, sink, gate, gate_ld,
+                                softcap)
     if nd < batch.n_tokens:
         ops.attention_prefill_ex(q, lane.k, lane.v, out, batch.seq_q_start[nd:], batch.seq_q_len[nd:],
                                  batch.seq_ctx_len[nd:], nd, max(batch.q_len[nd:]), table, lane.page_size, n_heads,
                                  need.n_kv_heads, need.head_dim, scale, window, vd, in_k, keep_first, sink, gate,
-                                 gate_ld)
+                                 gate_ld, softcap)
 
 
 _SINK_NAMES = {"q": "q", "k": "k", "v": "v", "g": "g", "o": "o", "sink": "sink"}
@@ -245,7 +247,7 @@ class SinkAttention(AttentionMixer):
 
 
 _NORMED_NAMES = {"q": "q", "k": "k", "v": "v", "o": "o", "q_bias": "q.b", "k_bias": "k.b", "q_norm": "q.norm",
-                 "k_norm": "k.norm"}
+                 "k_norm": "k.norm", "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv"}
 
 
 @register_mixer("normed_attention")
@@ -259,15 +261,21 @@ class NormedAttention(Mixer):
       heads) or None;
     * ``query_temperature``: ``{"coef", "every"}`` - the query at position p is multiplied by
       ``1 + coef ln(floor((p + 1) / every) + 1)``;
+    * ``conv``: taps of a causal convolution over time on every channel of q, k and v, directly behind the
+      projections (0: none; no bias, no activation); the last taps-1 projected rows are state of the request;
     * ``rotary``: ``{"dims", "base", "scaling"}`` - half-split pairs over the first ``dims`` channels of a head;
-      ``scaling`` None, ``{"factor"}`` (every frequency divided by it) or ``{"factor", "original", "fast",
-      "slow"}`` (the stretched table, cosine and sine times ``0.1 ln(factor) + 1``);
+      ``scaling`` None, ``{"factor"}`` (every frequency divided by it), ``{"factor", "original", "fast",
+      "slow"}`` (the stretched table, cosine and sine times ``0.1 ln(factor) + 1``) or ``{"factor", "original",
+      "low", "high"}`` (long waves divided by it, see ``rope.banded_inverse_wavelengths``);
     * ``values``: ``"own"`` (a value projection, ``v_head_dim`` wide per head) or ``"keys"`` (the keys as
       projected, with their bias, before norm and rotation);
     * ``rotate_values``: the value of position j is turned by j over all its channels (half-split pairs, pair m
       by ``j * base^(-2m/v_head_dim)``, no scaling) before it is cached, and a head's output at position i is
       turned back by i;
     * ``softmax_scale``, ``softcap`` (``cap * tanh(score / cap)``), ``window`` (0: causal);
+    * ``sink``: a number whose exponential joins every softmax denominator (None: none; 0 adds one);
+    * ``shares_cache``: the layer has queries only and reads the keys and values of the layer it names in the
+      schedule, as that layer's pages hold them;
     * ``out_f32``: the output projection is written in 32-bit."""
 
     graph_safe = True
@@ -289,6 +297,9 @@ class NormedAttention(Mixer):
         self.eps = float(p.get("eps", 1e-6))
         self.rotate_values = bool(p.get("rotate_values", False))
         self.out_f32 = bool(p.get("out_f32", False))
+        self.taps = int(p.get("conv", 0) or 0)
+        self.sink_value = p.get("sink")
+        self.shares_cache = bool(p.get("shares_cache", False))
         self.names = dict(_NORMED_NAMES, **(p.get("names") or {}))
         if self.values not in ("own", "keys"):
             raise ValueError(f"normed_attention: values must be 'own' or 'keys', got '{self.values}'")
@@ -304,14 +315,20 @@ class NormedAttention(Mixer):
             raise ValueError("normed_attention: values that are the keys have the keys' size")
         if self.rotate_values and self.vd % 2:
             raise ValueError("normed_attention: rotated values need an even v_head_dim")
-        from .rope import inverse_wavelengths, stretched_inverse_wavelengths
+        if self.taps < 0 or (self.taps and (self.values != "own" or self.bias)):
+            raise ValueError("normed_attention: a convolution goes with own values and without biases")
+        if self.shares_cache and (self.values != "own" or self.rotate_values or self.bias or self.qk_norm == "whole"):
+            raise ValueError("normed_attention: a layer that reads another's cache has queries and their norm per head only")
+        from .rope import banded_inverse_wavelengths, inverse_wavelengths, stretched_inverse_wavelengths
         rot = p.get("rotary") or {}
         self.rot = int(rot.get("dims", 0) or 0)
         if self.rot % 2 or self.rot > self.hd:
             raise ValueError(f"normed_attention: rotary dims {self.rot} must be even and at most head_dim")
         base, sc = float(rot.get("base", 10000.0)), rot.get("scaling") or None
         self.magnitude = 1.0
-        if sc and "original" in sc:
+        if sc and "low" in sc:
+            inv_f, inv_d = banded_inverse_wavelengths(self.rot, base, sc, runtime.device)
+        elif sc and "original" in sc:
             inv_f, inv_d, self.magnitude = stretched_inverse_wavelengths(self.rot, base, sc, runtime.device)
         else:
             inv_f, inv_d = inverse_wavelengths(self.rot, base, runtime.device)
@@ -323,13 +340,26 @@ class NormedAttention(Mixer):
         if self.rotate_values:
             vf, vd = inverse_wavelengths(self.vd, base, runtime.device)
             self.vinv_f, self.vinv_d = vf, (vd if runtime.precise else None)
-        self.w_in = self.w_o = self.b_in = self.q_w = self.k_w = None
+        self.w_in = self.w_o = self.b_in = self.q_w = self.k_w = self.conv_w = self.sink = None
 
     def _n(self, role: str) -> str:
         return self.prefix + self.names[role]
 
     def _roles(self):
+        if self.shares_cache:
+            return ("q",)
         return ("q", "k") + (("v",) if self.values == "own" else ())
+
+    @property
+    def n_own_kv(self) -> int:
+        """Key/value heads among the layer's own projections."""
+        return 0 if self.shares_cache else self.n_kv
+
+    @property
+    def conv_floats(self) -> int:
+        """Numbers of convolution state per request, a multiple of four."""
+        n = (self.taps - 1) * (self.n_heads * self.hd + self.n_own_kv * (self.hd + self.vd)) if self.taps > 1 else 0
+        return n + -n % 4
 
     def tensor_specs(self) -> Dict[str, TensorSpec]:
         nq, nk, nv = self.n_heads * self.hd, self.n_kv * self.hd, self.n_kv * self.vd
@@ -342,7 +372,10 @@ class NormedAttention(Mixer):
         if self.qk_norm:
             head = self.qk_norm == "head"
             specs[self._n("q_norm")] = TensorSpec((self.hd if head else nq,), role="vector")
-            specs[self._n("k_norm")] = TensorSpec((self.hd if head else nk,), role="vector")
+            if not self.shares_cache:
+                specs[self._n("k_norm")] = TensorSpec((self.hd if head else nk,), role="vector")
+        if self.taps:
+            specs.update({self._n(r + "_conv"): TensorSpec((rows[r], self.taps), role="vector") for r in self._roles()})
         return specs
 
     def bind(self, tensors) -> None:
@@ -356,53 +389,56 @@ class NormedAttention(Mixer):
             self.b_in = torch.cat(b).contiguous()
         if self.qk_norm:
             self.q_w = tensors[self._n("q_norm")].to(f32).contiguous()
-            self.k_w = tensors[self._n("k_norm")].to(f32).contiguous()
+            # a layer without keys has no weight for them; the kernel is given the queries' and never applies it
+            self.k_w = self.q_w if self.shares_cache else tensors[self._n("k_norm")].to(f32).contiguous()
+        if self.taps:
+            self.conv_w = torch.cat([tensors[self._n(r + "_conv")].to(f32) for r in self._roles()], dim=0).contiguous()
+        if self.sink_value is not None:
+            self.sink = torch.full((self.n_heads,), float(self.sink_value), dtype=f32, device=self.w_in.device)
 
     def weight_bytes(self) -> int:
         return (self.w_in.numel() + self.w_o.numel()) * self.w_in.element_size()
 
     def cache_need(self):
-        return PagedKV(self.n_kv, self.hd, self.window, v_head_dim=0 if self.vd == self.hd else self.vd)
+        kv = PagedKV(self.n_kv, self.hd, self.window, v_head_dim=0 if self.vd == self.hd else self.vd)
+        return (kv, FixedState((self.conv_floats,), tag="qkv_conv")) if self.conv_floats else kv
+
+    def _prepare(self, proj, batch, cache, state, q, writes_cache: bool) -> None:
+        """Convolution, biases, norms and rotations of the projections; queries to ``q``, keys and values into
+        their pages."""
+        table, kv = batch.block_table(cache.group), self.n_own_kv
+        per_head = self.qk_norm == "head"
+        writes_cache = writes_cache and not self.shares_cache
+        if self.taps:
+            plain = (self.qk_norm != "whole" and not self.rotate_values and self.temp_coef == 0.0 and self.magnitude == 1.0
+                     and (writes_cache or kv == 0))
+            if plain and ops.qkv_conv_ok(self.hd, self.vd, self.taps, proj.shape[1], self.rot):
+                ops.qkv_conv(proj, self.n_heads, kv, self.hd, self.vd, self.rot, self.eps, self.conv_w, self.q_w,
+                             self.k_w if kv else None, self.inv_f, self.inv_d, state, batch, table, cache.page_size, q,
+                             cache.k, cache.v)
+                return
+            y = self.rt.buffer("nattn.conv", tuple(proj.shape), torch.float32)
+            # a convolution of one tap keeps nothing, but its kernel wants an address
+            ops.conv_act(proj, proj.shape[1], self.conv_w, None, False, state if state is not None else proj, 0, batch, y)
+            proj = y
+        ops.qk_norm_rope(proj, self.n_heads, kv, self.hd, self.vd, self.rot, self.values == "keys", self.eps,
+                         self.magnitude, self.b_in, self.q_w, self.k_w, self.inv_f, self.inv_d, self.vinv_f, self.vinv_d,
+                         batch, table, cache.page_size, q, cache.k, cache.v, writes_cache, per_head,
+                         self.temp_coef, self.temp_every)
 
     def forward(self, x, batch, cache, writes_cache: bool = True):
         rt, T = self.rt, x.shape[0]
+        cache, state = cache if isinstance(cache, tuple) else (cache, None)
         # the projections feed 32-bit norms: they are written in 32-bit and rounded once, after norm and rotation
         proj = rt.linear(x, self.w_in, rt.buffer("nattn.in", (T, self.w_in.shape[0]), torch.float32))
         q = rt.buffer("nattn.q", (T, self.n_heads * self.hd))
-        table = batch.block_table(cache.group)
-        ops.qk_norm_rope(proj, self.n_heads, self.n_kv, self.hd, self.vd, self.rot, self.values == "keys", self.eps,
-                         self.magnitude, self.b_in, self.q_w, self.k_w, self.inv_f, self.inv_d, self.vinv_f, self.vinv_d,
-                         batch, table, cache.page_size, q, cache.k, cache.v, writes_cache, self.qk_norm == "head",
-                         self.temp_coef, self.temp_every)
+        self._prepare(proj, batch, cache, state.tensor if state is not None else None, q, writes_cache)
         o = rt.buffer("nattn.o", (T, self.n_heads * self.vd))
-        if not (self.window or self.softcap) and self.vd == self.hd and self.hd % 16 == 0 and self.hd <= 256:
+        if not (self.window or self.softcap or self.sink is not None) and self.vd == self.hd and self.hd % 16 == 0 and self.hd <= 256:
             paged_attention(rt, batch, q, cache, o, self.n_heads, self.scale, 0)       # nothing beyond the plain kernels
         else:
-            softcap_attention(rt, batch, q, cache, o, self.n_heads, self.scale, self.window, self.softcap)
+            options_paged_attention(rt, batch, q, cache, o, self.n_heads, self.scale, self.window, sink=self.sink,
+                                    softcap=self.softcap)
         if self.rotate_values:
             ops.rotate_rows(o, self.n_heads, self.vd, self.vd, batch.positions, self.vinv_f, self.vinv_d, -1.0)
         return rt.linear(o, self.w_o, rt.buffer("nattn.delta", (T, self.hidden), torch.float32 if self.out_f32 else None))
-
-
-def softcap_attention(rt, batch, q, lane, out, n_heads: int, scale: float, window: int, softcap: float) -> None:
-    """Attention over ``lane`` (values of their own width in a pool of their own) with a window and a soft cap
-    on the scaled scores; kernels chosen as in ``options_paged_attention``."""
-    need = lane.need
-    table = batch.block_table(lane.group)
-    vd = need.value_dim
-    if q.dtype != torch.bfloat16 or not ops.attention_tc_ok(need.head_dim, vd, lane.page_size):
-        ops.attention_generic_ex(q, lane.k, lane.v, out, batch.positions, batch.seq_of_token, table, lane.page_size,
-                                 n_heads, need.n_kv_heads, need.head_dim, scale, window, vd, vd, 0, None, None, 0,
-                                 softcap)
-        return
-    nd = batch.n_decode
-    if nd > 0:
-        n_o, n_ml = ops.attention_decode_scratch(nd, n_heads, need.head_dim, batch.max_ctx, window)
-        ops.attention_decode_ex(q[:nd], lane.k, lane.v, out[:nd], rt.buffer("attn.part_o", (n_o,), torch.float32),
-                                rt.buffer("attn.part_ml", (n_ml,), torch.float32), batch.positions[:nd],
-                                batch.seq_of_token[:nd], table, lane.page_size, n_heads, need.n_kv_heads,
-                                need.head_dim, scale, window, batch.max_ctx, vd, False, 0, None, None, 0, softcap)
-    if nd < batch.n_tokens:
-        ops.attention_prefill_ex(q, lane.k, lane.v, out, batch.seq_q_start[nd:], batch.seq_q_len[nd:],
-                                 batch.seq_ctx_len[nd:], nd, max(batch.q_len[nd:]), table, lane.page_size, n_heads,
-                                 need.n_kv_heads, need.head_dim, scale, window, vd, False, 0, None, None, 0, softcap)

@@ -203,6 +203,18 @@ class NormedPair:
     eps: float
 
 
+@dataclass(frozen=True)
+class PostNormed:
+    """A sublayer's output still to be normalised and then added to the stream:
+    ``x += norm(value) * weight`` (``kind``: ``"rms"`` or ``"layer"``).  The norm that reads the stream next
+    does both in its own kernel."""
+
+    value: Any
+    weight: Any
+    kind: str
+    eps: float
+
+
 # --------------------------------------------------------------------------- interfaces
 
 class Part:

@@ -103,6 +103,33 @@ class ParallelSharedNormBlock(Block):
         return residual, DeltaPair(d1, d2)
 
 
+@register_block("sandwich_norm")
+class SandwichNormBlock(Block):
+    """A norm before and a norm behind each sublayer: ``x += norm1b(mixer(norm1(x)))``, then (if the layer has a
+    feed-forward) ``x += norm2b(feed_forward(norm2(x)))``.  The norms behind the sublayers stand in the roles
+    ``mixer_post_norm`` and ``feed_forward_post_norm``; they and the norms before must be parts with
+    ``pending`` (``rmsnorm`` and ``layernorm``).  A sublayer's output travels on un-normalised and the norm that
+    reads the stream next (the layer's second one, the next layer's first one, the final one) does the whole
+    write: two kernels a layer for four norms and two adds."""
+
+    roles = ("mixer", "mixer_norm", "mixer_post_norm")
+
+    def __init__(self, by_role, runtime):
+        super().__init__(by_role, runtime)
+        self.mixer_post_norm = self.by_role["mixer_post_norm"]
+        self.feed_forward_post_norm = self.by_role.get("feed_forward_post_norm")
+        if self.feed_forward is not None and (self.feed_forward_norm is None or self.feed_forward_post_norm is None):
+            raise ValueError("sandwich_norm: a feed-forward needs a feed_forward_norm and a feed_forward_post_norm")
+
+    def forward(self, residual, pending, batch, cache, writes_cache: bool = True):
+        x = self.mixer_norm.add_forward(residual, pending)
+        pending = self.mixer_post_norm.pending(self.mixer.forward(x, batch, cache, writes_cache))
+        if self.feed_forward is not None:
+            x = self.feed_forward_norm.add_forward(residual, pending)
+            pending = self.feed_forward_post_norm.pending(self.feed_forward.forward(x, batch))
+        return residual, pending
+
+
 @register_block("postnorm_conv")
 class PostNormConvBlock(Block):
     """The norms sit on the sublayers' OUTPUTS and the sublayers read the stream itself through a short

@@ -3,7 +3,7 @@ optionally times a constant ``scale``)
 into the 32-bit residual stream (into every stream, where a model has several;
 optionally plus a sinusoidal position vector), and the output head (``logits = hn W^T`` with
 ``W = lm_head.weight`` when the checkpoint has it, else the embedding table,
-:346-350), computed only for the rows that were asked for, in float32."""
+:346-350), computed only for the rows that were asked for, in float32, optionally through a soft cap."""
 from __future__ import annotations
 
 from typing import Dict
@@ -72,6 +72,7 @@ class LinearHead(Part):
         self.name = self.prefix + str(params.get("tensor", "weight"))
         self.tied_to = params.get("tied_to")
         self.require_own = bool(params.get("require_own", False))
+        self.softcap = float(params.get("softcap") or 0.0)      # logits <- cap tanh(logits / cap); 0: as they are
         self.weight = None
 
     def tensor_specs(self) -> Dict[str, TensorSpec]:
@@ -92,4 +93,6 @@ class LinearHead(Part):
 
     def forward(self, x, out):
         """x [n, H] in the compute dtype -> float32 logits [n, V]."""
+        if self.softcap:
+            return self.rt.linear_softcap(x, self.weight, out, self.softcap)
         return self.rt.linear(x, self.weight, out)

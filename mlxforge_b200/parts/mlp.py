@@ -1,6 +1,7 @@
 """Dense feed-forwards.  Gated: ``down( act(gate(x)) * up(x) )`` with ``act`` = SiLU
 (src/model/decoder_model.cpp:277-282) or, as a parameter (``activation: "gelu_tanh"``), the tanh
-form of GELU; ``names`` maps the three roles to tensor names behind the prefix.  Gate and up are one matrix here, their
+form of GELU; ``activation: {"limit", "alpha", "up_offset"}`` is the clamped gate
+``g' sigmoid(alpha g') (u' + up_offset)`` of ``g' = min(g, limit)`` and ``u' = clamp(u, -limit, limit)``; ``names`` maps the three roles to tensor names behind the prefix.  Gate and up are one matrix here, their
 rows interleaved in groups of 8 (8 gate rows, then the matching 8 up rows) so a
 kernel that owns 16 consecutive output rows holds both halves of a product;
 when the intermediate size is no multiple of 8 the two are simply stacked.
@@ -9,6 +10,7 @@ Without a gate (``dense_mlp``): ``down( act(up(x)) )`` with ``act`` one of the s
 ``"relu2"``, the square of the rectified value; ``names`` maps the two roles to tensor names."""
 from __future__ import annotations
 
+import math
 from typing import Dict
 
 import torch
@@ -26,8 +28,14 @@ class SwiGLU(FeedForward):
         self.hidden = int(params["hidden_size"])
         self.inter = int(params["intermediate_size"])
         self.group = 8 if self.inter % 8 == 0 else self.inter
-        self.act = str(params.get("activation", "silu"))
-        ops.activation_code(self.act)
+        act = params.get("activation", "silu")
+        if isinstance(act, dict):
+            limit = act.get("limit")
+            self.act = ops.ClampedGate(math.inf if limit is None else float(limit), float(act.get("alpha", 1.702)),
+                                       float(act.get("up_offset", 1.0)))
+        else:
+            self.act = str(act)
+            ops.activation_code(self.act)
         n = params.get("names") or {}
         self.names = {"gate": n.get("gate", "gate_proj.weight"), "up": n.get("up", "up_proj.weight"),
                       "down": n.get("down", "down_proj.weight")}

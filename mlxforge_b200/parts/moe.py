@@ -5,7 +5,8 @@ Router (32-bit), by ``scoring``: ``s = sigmoid(Wr x)`` or ``s = softmax(Wr x)`` 
 The ``n_experts`` experts may form ``n_groups`` equal groups of neighbours; a group's score is the sum of
 its two largest ``s``, and only experts of the ``keep_groups`` best groups can be chosen (``n_groups`` = 0:
 any expert).  Each token uses the ``top`` allowed experts with the largest ``s`` (plus ``choice_bias``, a
-tensor with one number per router output that steers the choice and nothing else), weighted by
+tensor with one number per router output that steers the choice and nothing else; ``logit_bias`` names one
+that is added to the logits themselves), weighted by
 ``s * route_scale`` (not renormalised); ties go to the lower index.  Expert ``e``:
 
     g = min(Wg_e x, limit) ;  u = clamp(Wu_e x, -limit, limit) ;  y = Wd_e (g sigmoid(alpha g) (u + up_offset))
@@ -68,6 +69,7 @@ class RoutedExperts(FeedForward):
         if self.expert_act is not None:
             ops.activation_code(self.expert_act)
         self.choice_bias_name = p.get("choice_bias")
+        self.logit_bias_name = p.get("logit_bias")
         self.shared_gate_name = p.get("shared_gate")
         self.names = dict(_NAMES, **(p.get("names") or {}))
         if self.scoring not in ("sigmoid", "softmax"):
@@ -87,7 +89,7 @@ class RoutedExperts(FeedForward):
             raise ValueError("routed_experts: a shared gate without a shared branch")
         # tokens from which the sorted, tiled path is taken (bfloat16 only)
         self.grouped_min_tokens = int(p.get("grouped_min_tokens", 64))
-        self.w_router = self.w_gu = self.w_down = self.choice_bias = None
+        self.w_router = self.w_gu = self.w_down = self.choice_bias = self.logit_bias = None
 
     @property
     def n_outputs(self) -> int:
@@ -106,6 +108,8 @@ class RoutedExperts(FeedForward):
             specs[self._e(e, "down")] = TensorSpec((self.hidden, self.ff))
         if self.choice_bias_name:
             specs[self.prefix + self.choice_bias_name] = TensorSpec((self.n_outputs,), role="vector")
+        if self.logit_bias_name:
+            specs[self.prefix + self.logit_bias_name] = TensorSpec((self.n_outputs,), role="vector")
         if self.shared_gate_name:
             specs[self.prefix + self.shared_gate_name] = TensorSpec((1, self.hidden))
         if self.shared is not None:
@@ -128,6 +132,8 @@ class RoutedExperts(FeedForward):
             self.w_down = torch.zeros((0, self.hidden, self.ff), dtype=dt, device=self.w_router.device)
         if self.choice_bias_name:
             self.choice_bias = tensors[self.prefix + self.choice_bias_name].to(torch.float32).contiguous()
+        if self.logit_bias_name:
+            self.logit_bias = tensors[self.prefix + self.logit_bias_name].to(torch.float32).contiguous()
         if self.shared is not None:
             self.shared.bind(tensors)
 
@@ -145,7 +151,7 @@ class RoutedExperts(FeedForward):
         ids = self.rt.buffer("moe.ids", (T, self.top), torch.int32)
         weights = self.rt.buffer("moe.weights", (T, self.top), torch.float32)
         ops.moe_route(z, self.n_groups, self.keep, self.top, self.route_scale, ids, weights, self.n_outputs,
-                      self.scoring == "softmax", self.choice_bias, self.renormalize)
+                      self.scoring == "softmax", self.choice_bias, self.renormalize, self.logit_bias)
         return ids, weights, z
 
     def _combine(self, y, weights, slot_of, out, slices, ids, x, z, shared):

@@ -8,7 +8,12 @@ is the same product).  ``post_add`` is the norm on a sublayer's OUTPUT: ``residu
 
 A layer whose branches run side by side on one residual hands on two deltas at once
 (``DeltaPair``) and wants two norms of the same sum: ``RMSNorm.pair_forward`` adds both deltas
-and applies both weights in one kernel."""
+and applies both weights in one kernel.
+
+``layernorm`` takes the mean off first and divides by the root of the mean squared deviation; it has a
+weight and no bias.  A norm on a sublayer's output hands that output on with ``pending`` (a
+``PostNormed``); the next norm of the stream, of either kind, normalises it, adds it and norms the sum
+in one kernel."""
 from __future__ import annotations
 
 from typing import Dict
@@ -16,7 +21,7 @@ from typing import Dict
 import torch
 
 from ..csrc import ops
-from .base import DeltaPair, Norm, NormedPair, ScaledPair, TensorSpec, register_norm
+from .base import DeltaPair, Norm, NormedPair, PostNormed, ScaledPair, TensorSpec, register_norm
 
 
 @register_norm("rmsnorm")
@@ -57,11 +62,18 @@ class RMSNorm(Norm):
         else:
             ops.postnorm_add(residual, y, 1.0, None, 0.0, self.weight, self.eps)
 
+    def pending(self, y) -> PostNormed:
+        """``y``, a sublayer's output that this norm stands behind, as what is still to be added to the stream."""
+        return PostNormed(y, self.weight, "rms", self.eps)
+
     def add_forward(self, residual, delta, out=None, rows=None):
         n = residual.shape[0] if rows is None else rows.shape[0]
         if out is None:
             out = self.rt.buffer("norm.out", (n, self.size))
-        if isinstance(delta, DeltaPair):
+        if isinstance(delta, PostNormed):
+            ops.post_norm(residual, delta.value, delta.weight, delta.kind, delta.eps, self.weight, "rms", self.eps, out,
+                          rows)
+        elif isinstance(delta, DeltaPair):
             ops.add_rmsnorm_pair(residual, delta.first, delta.second, self.weight, None, self.eps, out, None, rows)
         else:
             ops.add_rmsnorm(residual, delta, self.weight, self.eps, out, rows)
@@ -79,6 +91,47 @@ class RMSNorm(Norm):
         ops.add_rmsnorm_pair(residual, pair.first, pair.second, self.weight, other.weight if other is not None else None,
                              self.eps, out1, out2)
         return out1, out2
+
+
+@register_norm("layernorm")
+class LayerNorm(Norm):
+    """``(x - mean) / sqrt(variance + eps) * w`` over the last axis, no bias, the variance being the mean of the
+    squared deviations; all of it in 32-bit."""
+
+    graph_safe = True
+
+    def __init__(self, params, prefix, runtime):
+        super().__init__(params, prefix, runtime)
+        self.size = int(params["size"])
+        self.eps = float(params["eps"])
+        self.name = self.prefix + str(params.get("tensor", "weight"))
+        self.weight = None
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        return {self.name: TensorSpec((self.size,), role="vector")}
+
+    def bind(self, tensors) -> None:
+        self.weight = tensors[self.name].to(torch.float32).contiguous()
+
+    def weight_bytes(self) -> int:
+        return self.size * 4
+
+    def forward(self, x, out=None):
+        return self.add_forward(x, None, out)
+
+    def pending(self, y) -> PostNormed:
+        return PostNormed(y, self.weight, "layer", self.eps)
+
+    def add_forward(self, residual, delta, out=None, rows=None):
+        n = residual.shape[0] if rows is None else rows.shape[0]
+        if out is None:
+            out = self.rt.buffer("norm.out", (n, self.size))
+        if isinstance(delta, PostNormed):
+            ops.post_norm(residual, delta.value, delta.weight, delta.kind, delta.eps, self.weight, "layer", self.eps, out,
+                          rows)
+        else:
+            ops.post_norm(residual, delta, None, None, 0.0, self.weight, "layer", self.eps, out, rows)
+        return out
 
 
 @register_norm("group_rmsnorm")

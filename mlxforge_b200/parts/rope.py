@@ -133,6 +133,27 @@ def stretched_inverse_wavelengths(rotary_dim: int, base: float, scaling, device)
     return (torch.from_numpy(inv.astype(np.float32)).to(device), torch.from_numpy(inv).to(device), magnitude)
 
 
+def banded_inverse_wavelengths(rotary_dim: int, base: float, scaling, device):
+    """Inverse wavelengths ``w = base^(-2i/dims)`` of a rotation whose long waves are slowed down (the schedule of
+    Llama 3.1): (float32 tensor, float64 tensor).  ``scaling`` has ``factor``, ``low``, ``high`` and ``original``
+    (the trained context).  A wave ``l = 2 pi / w`` shorter than ``original / high`` keeps ``w``, one longer than
+    ``original / low`` gets ``w / factor``, and between them, with ``s = (original / l - low) / (high - low)``,
+    it is ``(1 - s) w / factor + s w``.  ``scaling`` None: the plain table.  Worked out in double."""
+    if rotary_dim < 0 or rotary_dim % 2:
+        raise ValueError(f"rotary_dim must be even and not negative, got {rotary_dim}")
+    inv = np.power(float(base), -2.0 * np.arange(rotary_dim // 2, dtype=np.float64) / max(rotary_dim, 1))
+    if scaling:
+        factor, original = float(scaling["factor"]), float(scaling["original"])
+        low, high = float(scaling["low"]), float(scaling["high"])
+        if not (factor > 0 and original > 0 and low > 0 and high > 0):
+            raise ValueError("banded rotation: factor, original, low and high must be positive")
+        wave = 2.0 * np.pi / inv
+        s = (original / wave - low) / (high - low if high != low else 1.0)
+        blend = (1.0 - s) * inv / factor + s * inv
+        inv = np.where(wave < original / high, inv, np.where(wave > original / low, inv / factor, blend))
+    return (torch.from_numpy(inv.astype(np.float32)).to(device), torch.from_numpy(inv).to(device))
+
+
 @register_position("rotary")
 class Rotary(PositionEncoding):
     graph_safe = True
