@@ -196,7 +196,7 @@ def mixture(h, w, mlp):
         rows = np.nonzero(weights[:, e])[0]
         if len(rows):
             y[rows] += weights[rows, e, None] * clamped_feed_forward(h[rows], w[f"e{e}.gate"], w[f"e{e}.up"],
-                                                                     w[f"e{e}.down"], mlp["expert"]["limit"])
+                                                                     w[f"e{e}.down"], mlp["expert"].get("limit", np.inf))
     return y
 
 
@@ -228,8 +228,16 @@ def forward(cfg, w, tokens, layers_out=None):
         if mlp is not None:
             h, fw = layer_norm(x, lw["norm2"], eps), _under(lw, "mlp.")
             y = (mixture(h, fw, mlp) if mlp["kind"] == "moe"
-                 else clamped_feed_forward(h, fw["gate"], fw["up"], fw["down"], mlp["limit"]))
+                 else clamped_feed_forward(h, fw["gate"], fw["up"], fw["down"], mlp.get("limit", np.inf)))
             x = x + layer_norm(_r(y), lw["norm2b"], eps)
         if layers_out is not None:
             layers_out.append(x.copy())
     return soft_cap(lin(layer_norm(x, w["final.norm"], eps), w["embed"]), cfg.get("logit_softcap"))
+
+
+def generate(cfg, w, tokens, n):
+    """``n`` greedy tokens after ``tokens``."""
+    seq = list(tokens)
+    for _ in range(n):
+        seq.append(int(np.argmax(forward(cfg, w, seq)[-1])))
+    return seq[len(tokens):]

@@ -48,7 +48,7 @@ def rand(rng, *shape, std=1.0):
 
 
 class Harness:
-    """A runtime, a cache with one lane of the given need and the runner's metadata builder."""
+    """A runtime, a cache with one lane of the given need (or one of each of several) and the runner's metadata builder."""
 
     def __init__(self, dtype, need, lengths=LENGTHS, steps=STEPS, page_size=16, max_tokens=512):
         import torch
@@ -57,9 +57,12 @@ class Harness:
         from mlxforge_b200.engine.step import ModelRunner
         from mlxforge_b200.parts.base import PagedKV
         self.rt = Runtime(tdt(dtype))
-        paged = isinstance(need, PagedKV)
-        layout = CacheLayout(paged=(GroupLayout(need, 1),) if paged else (), state=() if paged else (GroupLayout(need, 1),),
-                             item_lane=(("paged" if paged else "state", 0, 0),))
+        needs = need if isinstance(need, tuple) else (need,)
+        paged = tuple(n for n in needs if isinstance(n, PagedKV))
+        state = tuple(n for n in needs if not isinstance(n, PagedKV))
+        lanes = tuple(("paged", paged.index(n), 0) if isinstance(n, PagedKV) else ("state", state.index(n), 0) for n in needs)
+        layout = CacheLayout(paged=tuple(GroupLayout(n, 1) for n in paged), state=tuple(GroupLayout(n, 1) for n in state),
+                             item_lane=(lanes if isinstance(need, tuple) else lanes[0],))
         self.cache = CacheManager(layout, page_size=page_size, max_tokens=max_tokens, max_seqs=4, dtype=tdt(dtype),
                                   device="cuda")
         for pool in self.cache._k + self.cache._v:
