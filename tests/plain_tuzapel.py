@@ -23,6 +23,7 @@ from __future__ import annotations
 import numpy as np
 
 ROUND = None          # a function applied to activations where a bfloat16 engine rounds; None = exact
+GAPS = None           # a list that receives, per router and token, how much the last chosen logit leads the next
 
 
 def _r(x):
@@ -183,6 +184,9 @@ def clamped_feed_forward(h, gate, up, down, limit):
 def choose_experts(z, top):
     """z [T, E] -> weights [T, E], zero where an expert is not chosen."""
     out = np.zeros_like(z)
+    if GAPS is not None and top < z.shape[1]:
+        s = -np.sort(-z, axis=-1)
+        GAPS.extend(s[:, top - 1] - s[:, top])
     for t in range(z.shape[0]):
         best = np.argsort(-z[t], kind="stable")[:top]
         out[t, best] = softmax(z[t, best])

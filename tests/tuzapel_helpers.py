@@ -161,24 +161,36 @@ def tensor_shapes(cfg):
 
 def random_weights(cfg, seed, qk_gain=1.0):
     """float32 arrays, exact in bfloat16.  ``qk_gain`` scales the query and key norm weights so that the softmax
-    is peaked and a wrong or missing key shows."""
+    is peaked and a wrong or missing key shows.
+
+    A choice of experts that hangs on the last bit would flip under rounding and hide every other difference, so
+    the first channels of the stream hold a code of the token (one of a few classes) that no sublayer writes to,
+    and the routers read mostly that: which experts a token takes varies from token to token, by clear margins."""
     rng = np.random.default_rng(seed)
     w = {}
+    K = min(6, cfg["width"] // 4)
     for name, shape in tensor_shapes(cfg):
         n = lambda std, mean=0.0: (mean + rng.standard_normal(shape) * std).astype(np.float32)
         leaf = name.split(".")[-1]
         if name == "embed":
-            a = n(0.7, 0.1)
-        elif leaf in ("norm1", "norm1b", "norm2", "norm2b") or name == "final.norm":
+            a = n(0.5)
+            a[:, :K] = 0.0
+            a[np.arange(len(a)), np.arange(len(a)) % K] = 2.0
+        elif leaf in ("norm1b", "norm2b"):
+            a = n(0.1, 0.5)
+            a[:K] = 0.0
+        elif leaf in ("norm1", "norm2") or name == "final.norm":
             a = n(0.15, 1.0)
         elif leaf == "norm":
             a = n(0.1, 1.0) * np.float32(qk_gain if name.split(".")[-2] in ("q", "k", "dq") else 1.0)
         elif leaf == "conv":
             a = n(0.5)
         elif leaf == "b":
-            a = n(0.5)
+            a = n(0.15)
         elif leaf == "router":
-            a = n(2.0 / np.sqrt(shape[-1]))
+            a = n(0.1 / np.sqrt(shape[-1]))
+            for c in range(K):
+                a[:, c] = 0.4 * (rng.permutation(shape[0]) - (shape[0] - 1) / 2)
         else:
             a = n(1.2 / np.sqrt(shape[-1]))
         w[name] = bf16_round(a.astype(np.float32))
