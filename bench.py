@@ -543,6 +543,16 @@ def kernel_work(name, a, k, info):
     if name == "gated_norm":
         x, out = a[0], a[5]
         return (_nbytes(x) + out.numel() * 4 + _nbytes(out), 0, 0)
+    if name == "post_norm":
+        resid, y, out, rows = a[0], a[1], a[8], (a[9] if len(a) > 9 else None)
+        n = out.shape[0]
+        return (n * resid.shape[1] * 4 * (2 if y is not None and rows is None else 1) + _nbytes(out)
+                + (n * y.shape[1] * y.element_size() if y is not None else 0), 0, 0)
+    if name == "qkv_conv":
+        proj, n_kv, hd, vd, q_out = a[0], a[2], a[3], a[4], a[16]
+        return (_nbytes(proj, q_out) + T * n_kv * (hd + vd) * q_out.element_size(), 0, 0)
+    if name == "soft_cap":
+        return (2 * _nbytes(a[0]), 0, 0)
     if name == "low_rank":
         wt, out = a[2], a[4]
         return (_nbytes(wt, out) + T * wt.shape[0] * 4, 0, 2.0 * T * wt.shape[0] * wt.shape[1])
@@ -996,6 +1006,60 @@ def run_takavik(args) -> int:
                                  ("notirax_equal_size", takavik_notirax_like(z), NOTIRAX_KERNELS, z["context"])))
 
 
+# ---------------------------------------------------------------------------- --workload tuzapel
+# The Tuzapel design at sizes that resemble a real model's layers, beside the two closest existing models at equal
+# size (width, layers, vocabulary, heads, head sizes, ranks, window): a Luzinex decoder with attention within a window
+# beside a learned sink and latent attention, all with gated dense feed-forwards, and a Rabapel decoder (latent
+# attention, every other layer a mixture of gated experts of the same number and width).
+TUZAPEL_SIZES = {
+    "s": dict(width=1024, layers=6, vocab=32768, heads=8, kv=2, dim=128, rot=64, window=1024, conv=4, l_heads=8, l_dim=64,
+              l_rot=32, l_vdim=64, q_rank=384, kv_rank=128, ff=4096, experts=32, top=4, expert_ff=512, context=4096),
+    "m": dict(width=2048, layers=6, vocab=32768, heads=16, kv=4, dim=128, rot=64, window=2048, conv=4, l_heads=16, l_dim=64,
+              l_rot=32, l_vdim=64, q_rank=768, kv_rank=192, ff=8192, experts=32, top=4, expert_ff=1024, context=4096),
+}
+TUZAPEL_KERNELS = ("embed", "post_norm", "qkv_conv", "conv_act", "qk_norm_rope", "latent_prepare", "latent_query",
+                   "head_linear", "head_linear_mma", "attention_prefill_ex", "attention_decode_ex", "attention_generic_ex",
+                   "moe_route", "moe_rows", "moe_combine", "moe_sort", "moe_grouped_up", "moe_grouped_down",
+                   "moe_gather_rows", "moe_activation", "_grouped_mm", "swiglu", "soft_cap", "stream_linear", "gemm_bf16")
+
+
+def tuzapel_config(z):
+    attn = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5,
+            "conv": z["conv"], "mask": {"size": z["window"]},
+            "rot": {"base": 500000.0, "dims": z["rot"],
+                    "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": z["context"] // 2}}}
+    latent = {"heads": z["l_heads"], "dim": z["l_dim"], "rot_dim": z["l_rot"], "vdim": z["l_vdim"], "q_rank": z["q_rank"],
+              "kv_rank": z["kv_rank"], "scale": (z["l_dim"] + z["l_rot"]) ** -0.5, "rot": {"base": 50000.0, "dims": z["l_rot"]}}
+    dense = {"kind": "dense", "ff": z["ff"], "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"], "limit": 7.0}, "router": {"experts": z["experts"], "top": z["top"]}}
+    order = [("attention", attn, dense), ("latent_attention", latent, moe), ("attention", attn, moe),
+             ("attention", dict(attn, kv_from=2), dense), ("latent_attention", latent, dense),
+             ("attention", dict(attn, kv_from=2), moe)]
+    return {"architecture": "Tuzapel", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "logit_softcap": 30.0,
+            "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in order[:z["layers"]]]}
+
+
+def tuzapel_luzinex_like(z):
+    like = luzinex_config(dict(z, keep=0, r_heads=1, r_dim=16, r_vdim=16))
+    latent, attn = like["layers"][0]["mixer"], like["layers"][1]["mixer"]
+    mlp = like["layers"][0]["mlp"]
+    like["layers"] = [{"type": "latent_attention", "mixer": dict(latent), "mlp": mlp} if i % 3 == 1 else
+                      {"type": "attention", "mixer": dict(attn), "mlp": mlp} for i in range(z["layers"])]
+    return like
+
+
+def tuzapel_rabapel_like(z):
+    return rabapel_config(dict(z, heads=z["l_heads"], dim=z["l_dim"], rot=z["l_rot"], vdim=z["l_vdim"], identity=0,
+                               shared_ff=z["expert_ff"]))
+
+
+def run_tuzapel(args) -> int:
+    return run_beside(args, "tuzapel", TUZAPEL_SIZES,
+                      lambda z: (("tuzapel", tuzapel_config(z), TUZAPEL_KERNELS, 0),
+                                 ("luzinex_equal_size", tuzapel_luzinex_like(z), LUZINEX_KERNELS, 0),
+                                 ("rabapel_equal_size", tuzapel_rabapel_like(z), RABAPEL_KERNELS, 0)))
+
+
 # Kinds of launches that `--without` leaves out of a decode step, to see what each costs inside it.
 LEFT_OUT = ("norms", "rotation", "attention", "qkv", "o", "gate_up", "down", "head", "products")
 
@@ -1050,13 +1114,14 @@ def main() -> int:
     ap.add_argument("--without", default=None, choices=sorted(LEFT_OUT),
                     help="with --only decode: time the step with the launches of one kind left out (its results are "
                          "wrong; the difference to the full step is what that kind costs inside the step)")
-    ap.add_argument("--workload", default="headline", choices=["headline", "serving", "longctx", "notirax", "luzinex", "rabapel", "ledinex", "takavik"],
+    ap.add_argument("--workload", default="headline", choices=["headline", "serving", "longctx", "notirax", "luzinex", "rabapel", "ledinex", "takavik", "tuzapel"],
                     help="serving: 64 requests on the 3B shape; longctx: 8 x 16,384 tokens on the 8B shape; notirax / "
                          "luzinex: prefill and decode of that design beside the Llama decoder at equal size, per kernel; "
                          "rabapel: the same beside a Luzinex decoder of latent-attention layers at equal size; "
-                         "ledinex / takavik: the same beside a Notirax decoder at equal size")
+                         "ledinex / takavik: the same beside a Notirax decoder at equal size; tuzapel: the same beside a Luzinex "
+                         "and a Rabapel decoder at equal size")
     ap.add_argument("--size", default=None, choices=sorted(set(NOTIRAX_SIZES) | set(LUZINEX_SIZES) | set(RABAPEL_SIZES)),
-                    help="with --workload notirax, luzinex, rabapel, ledinex or takavik: one size only")
+                    help="with --workload notirax, luzinex, rabapel, ledinex, takavik or tuzapel: one size only")
     args = ap.parse_args()
     args.shape_given = args.shape is not None
     args.shape = args.shape or "1b"
@@ -1078,6 +1143,8 @@ def main() -> int:
         return run_ledinex(args)
     if args.workload == "takavik":
         return run_takavik(args)
+    if args.workload == "tuzapel":
+        return run_tuzapel(args)
     if args.workload != "headline":
         return run_workload(args)
 
