@@ -53,11 +53,14 @@ struct EpiConst {
   float limit, alpha, up_off;      // of the clamped gate
   float cap;                       // of the soft cap
 };
+// QUICK: for results that are rounded to bfloat16 (a division and an exponential of a few 32-bit ulps)
+template <bool QUICK = false>
 __device__ __forceinline__ float gated_product(float g, float u, int act, const EpiConst& k) {
   if (act == MF_GATE_CLAMPED) {
     g = fminf(g, k.limit);
     u = fminf(fmaxf(u, -k.limit), k.limit);
-    return g / (1.0f + expf(-k.alpha * g)) * (u + k.up_off);
+    const float s = QUICK ? __fdividef(g, 1.0f + __expf(-k.alpha * g)) : g / (1.0f + expf(-k.alpha * g));
+    return s * (u + k.up_off);
   }
   return gate_act(g, act) * u;
 }

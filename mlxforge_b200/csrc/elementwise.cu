@@ -360,7 +360,7 @@ __global__ void swiglu_bf16_g8_kernel(const uint4* __restrict__ gu, uint4* __res
 #pragma unroll
   for (int e = 0; e < 4; e++) {
     const float2 g = __bfloat1622float2(gp[e]), u = __bfloat1622float2(up[e]);
-    p[e] = __floats2bfloat162_rn(gated_product(g.x, u.x, act, ec), gated_product(g.y, u.y, act, ec));
+    p[e] = __floats2bfloat162_rn(gated_product<true>(g.x, u.x, act, ec), gated_product<true>(g.y, u.y, act, ec));
   }
   out[idx] = pk;
 }

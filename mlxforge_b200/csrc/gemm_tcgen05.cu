@@ -93,7 +93,7 @@ __device__ __forceinline__ unsigned pack_bf16(float lo, float hi) {
 constexpr int EPI_CLAMPED = 4 + MF_ACT_COUNT;
 template <int EPI> __device__ __forceinline__ float epi_gate(float g, float u, const EpiConst& ec) {
   constexpr int act = EPI == EPI_CLAMPED ? MF_GATE_CLAMPED : EPI == 3 ? MF_ACT_GELU_TANH : MF_ACT_SILU;
-  return gated_product(g, u, act, ec);
+  return gated_product<true>(g, u, act, ec);
 }
 
 // a sum on its way into a bfloat16 C: as it is (EPI 0) or through the activation EPI - 4 (EPI >= 4)

@@ -879,13 +879,13 @@ def qkv_conv(proj: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, v_dim: 
              block_table: torch.Tensor, page_size: int, q_out: torch.Tensor, k_pool: torch.Tensor,
              v_pool: torch.Tensor) -> None:
     """From 32-bit projections [queries | keys | values] (``n_kv`` 0: queries alone): the causal convolution
-    over time (``conv_w`` [channels, taps], the last taps-1 rows of every sequence at the start of its slot of
+    over time (``conv_w`` [taps, channels], a row per tap; the last taps-1 rows of every sequence at the start of its slot of
     ``state``, which move on), the norms per head (``q_w``, ``k_w`` [head_dim]; None: no norm), the rotation of
     half-split pairs, and the cache write."""
     _need_cuda(proj, conv_w, q_w, k_w, inv_f, inv_d, state, block_table, q_out, k_pool, v_pool)
-    T, taps = proj.shape[0], conv_w.shape[1]
-    if proj.dtype != torch.float32 or conv_w.shape[0] != n_heads * head_dim + n_kv * (head_dim + v_dim):
-        raise KernelError("qkv_conv: 32-bit projections and a row of taps per channel")
+    T, taps = proj.shape[0], conv_w.shape[0]
+    if proj.dtype != torch.float32 or conv_w.shape[1] != n_heads * head_dim + n_kv * (head_dim + v_dim):
+        raise KernelError("qkv_conv: 32-bit projections and a weight per tap and channel")
     if taps > 1 and (state is None or state.dtype != torch.float32):
         raise KernelError("qkv_conv: a convolution of several taps needs a state")
     check(library().mf_qkv_conv(proj.data_ptr(), proj.shape[1], dtype_code(q_out), T, n_heads, n_kv, head_dim, v_dim, rot,

@@ -13,10 +13,11 @@
 // rows of a sequence's projections stay in its state slot ([taps-1, channels] at `tail_off`), so a step
 // goes on from where the step before ended however the tokens were cut.
 //
-// A warp owns a head over a run of consecutive tokens: a lane holds two neighbouring channels of every
-// 64, the convolution's window stays in registers, so every input is read once; the cosines and sines
-// of the run's positions are worked out once for all heads of the block.  Everything is 32-bit
-// (angles in double where a float64 table is given) and is rounded once, on its way into q_out
+// A warp owns a head over a run of R consecutive tokens; a lane holds two neighbouring channels of every
+// 64.  The run's inputs are all fetched first (each once, the taps-1 before the run again), the taps are
+// applied in registers, and the places of the run's tokens in the pages are worked out by one lane each;
+// the cosines and sines of the run's positions are made once for all heads of the block.  Everything is
+// 32-bit (angles in double where a float64 table is given) and is rounded once, on its way into q_out
 // [T, n_heads * hd] and the pages.  Where every sequence of the step brings one token a head's warp is
 // the only reader of its columns of the slot and moves them on itself; else a second kernel does.
 #include "conv_tail.cuh"
@@ -41,23 +42,25 @@ __device__ __forceinline__ void store2(__nv_bfloat16* p, float a, float b) {
   *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
 }
 
-// NC: pieces of 64 channels a head has at most
-template <typename TO, int TAPS, int NC>
-__global__ void __launch_bounds__(WARPS * 32)
-qkv_conv_kernel(const float* __restrict__ proj, int ld, QkvConv p, const float* __restrict__ w, float* __restrict__ state,
-                long long state_stride, long long tail_off, const int* __restrict__ positions,
+constexpr int MAXT = 4;      // taps a lane holds; fewer are padded with zeros in front
+
+// R: tokens of a run; NC: pieces of 64 channels a head has at most
+template <typename TO, int R, int NC>
+__global__ void __launch_bounds__(WARPS * 32, 2)
+qkv_conv_kernel(const float* __restrict__ proj, int ld, QkvConv p, const float* __restrict__ w, int taps,
+                float* __restrict__ state, long long state_stride, long long tail_off, const int* __restrict__ positions,
                 const int* __restrict__ seq_of_token, const int* __restrict__ seq_q_start, const int* __restrict__ slots,
                 PagedView pk, PagedView pvv, TO* __restrict__ q_out, TO* __restrict__ k_pool, TO* __restrict__ v_pool,
-                int T, int run, int move_tail) {
-  extern __shared__ float qc_sm[];         // cos and sin of the run's positions, then a head's row per warp
+                int T, int move_tail) {
+  extern __shared__ float qc_sm[];         // cos and sin of the run's positions, then R rows of a head per warp
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int half = p.rot >> 1;
-  const int t0 = blockIdx.x * run, t1 = min(T, t0 + run);
+  const int t0 = blockIdx.x * R, n_run = min(R, T - t0);
   float* cs = qc_sm;
-  float* buf = qc_sm + run * p.rot + warp * (NC * 64);
+  float* buf = qc_sm + R * p.rot + warp * (R * NC * 64);
   pdl_launch();
   // positions, weights and tables are in place before the step's first kernel: no need to wait for them
-  for (int i = threadIdx.x; i < (t1 - t0) * half; i += blockDim.x) {
+  for (int i = threadIdx.x; i < n_run * half; i += blockDim.x) {
     const int tt = i / half, j = i - tt * half;
     float c, s;
     rotary_cs(positions[t0 + tt], j, p.inv_f, p.inv_d, c, s);
@@ -73,114 +76,134 @@ qkv_conv_kernel(const float* __restrict__ proj, int ld, QkvConv p, const float* 
   const int width = is_v ? p.vd : p.hd;
   const int col = is_q ? head * p.hd : is_v ? nq + nk + head * p.vd : nq + head * p.hd;
   const float* nw = is_v ? nullptr : is_q ? p.q_w : p.k_w;
-  float2 wt[NC][TAPS], norm_w[NC];
+  float2 wt[NC][MAXT], norm_w[NC];
 #pragma unroll
   for (int n = 0; n < NC; n++) {
     const int c = n * 64 + 2 * lane;
     norm_w[n] = make_float2(1.f, 1.f);
-    if (live && c < width) {
-      if (nw) norm_w[n] = make_float2(nw[c], nw[c + 1]);
+    const bool in = live && c < width;
+    if (in && nw) norm_w[n] = make_float2(nw[c], nw[c + 1]);
 #pragma unroll
-      for (int j = 0; j < TAPS; j++)
-        wt[n][j] = make_float2(w[(long long)(col + c) * TAPS + j], w[(long long)(col + c + 1) * TAPS + j]);
+    for (int j = 0; j < MAXT; j++) {
+      const int tap = j - (MAXT - taps);
+      wt[n][j] = in && tap >= 0 ? *reinterpret_cast<const float2*>(w + (long long)tap * C + col + c) : make_float2(0.f, 0.f);
     }
+  }
+  // lane i looks up token i of the run: its distance from the first token its sequence brings, its slot and
+  // where its row goes
+  int my_rel = 0, my_slot = 0;
+  long long my_dst = 0;
+  if (live && lane < n_run) {
+    const int t = t0 + lane, seq = seq_of_token[t];
+    my_rel = t - seq_q_start[seq];
+    my_slot = slots[seq];
+    my_dst = is_q ? (long long)t * nq + col : paged_offset(is_v ? pvv : pk, seq, positions[t], head);
   }
   __syncthreads();
   pdl_wait();
   if (!live) return;
-  float2 win[NC][TAPS];        // the last TAPS inputs of every channel, the newest last
+  // u[i + MAXT - 1] is token i of the run; what stands before it is used by the tokens of its own sequence only
+  float2 u[R + MAXT - 1][NC];
 #pragma unroll
-  for (int n = 0; n < NC; n++)
-#pragma unroll
-    for (int j = 0; j < TAPS; j++) win[n][j] = make_float2(0.f, 0.f);
-  for (int t = t0; t < t1; t++) {
-    const int seq = seq_of_token[t];
-    const int rel = t - seq_q_start[seq];
-    float* tail = TAPS > 1 ? state + (long long)slots[seq] * state_stride + tail_off : nullptr;
-    float2 y[NC];
-    float ss = 0.f;
+  for (int i = 0; i < R + MAXT - 1; i++) {
+    const int t = t0 + i - (MAXT - 1);
+    const bool row = t >= 0 && i - (MAXT - 1) < n_run && i >= MAXT - taps;
 #pragma unroll
     for (int n = 0; n < NC; n++) {
       const int c = n * 64 + 2 * lane;
-      y[n] = make_float2(0.f, 0.f);
-      if (c < width) {
-        if (t == t0 || rel == 0) {
+      u[i][n] = row && c < width ? *reinterpret_cast<const float2*>(proj + (long long)t * ld + col + c) : make_float2(0.f, 0.f);
+    }
+  }
 #pragma unroll
-          for (int j = 0; j < TAPS - 1; j++) {
-            const int back = TAPS - 1 - j;
-            win[n][j + 1] = rel - back >= 0
-                                ? *reinterpret_cast<const float2*>(proj + (long long)(t - back) * ld + col + c)
-                                : *reinterpret_cast<const float2*>(tail + (long long)(rel - back + TAPS - 1) * C + col + c);
-          }
-        }
+  for (int i = 0; i < R; i++) {
+    const int rel = __shfl_sync(0xffffffffu, my_rel, i);
+    float2 y[NC];
+    if (rel >= taps - 1) {           // every input is among the rows of this step
 #pragma unroll
-        for (int j = 0; j < TAPS - 1; j++) win[n][j] = win[n][j + 1];
-        win[n][TAPS - 1] = *reinterpret_cast<const float2*>(proj + (long long)t * ld + col + c);
+      for (int n = 0; n < NC; n++) {
+        y[n] = make_float2(0.f, 0.f);
 #pragma unroll
-        for (int j = 0; j < TAPS; j++) {
-          y[n].x = fmaf(wt[n][j].x, win[n][j].x, y[n].x);
-          y[n].y = fmaf(wt[n][j].y, win[n][j].y, y[n].y);
-        }
-        ss = fmaf(y[n].x, y[n].x, fmaf(y[n].y, y[n].y, ss));
-        if (TAPS > 1 && move_tail) {     // the sequence's only token: what was read, one place on
-#pragma unroll
-          for (int j = 0; j < TAPS - 1; j++)
-            *reinterpret_cast<float2*>(tail + (long long)j * C + col + c) = win[n][j + 1];
+        for (int j = 0; j < MAXT; j++) {
+          if (j < MAXT - taps) continue;          // a padded tap: another sequence's row may stand there
+          y[n].x = fmaf(wt[n][j].x, u[i + j][n].x, y[n].x);
+          y[n].y = fmaf(wt[n][j].y, u[i + j][n].y, y[n].y);
         }
       }
-    }
-    const int pos = positions[t];
-    if (is_v) {
-      TO* dst = v_pool + paged_offset(pvv, seq, pos, head);
+    } else {                         // the first tokens of a portion: the slot has what came before
+      float* tail = state + (long long)__shfl_sync(0xffffffffu, my_slot, i) * state_stride + tail_off + col;
 #pragma unroll
       for (int n = 0; n < NC; n++) {
         const int c = n * 64 + 2 * lane;
-        if (c < width) store2(dst + c, y[n].x, y[n].y);
+        y[n] = make_float2(0.f, 0.f);
+        float2 seen[MAXT];
+#pragma unroll
+        for (int j = 0; j < MAXT; j++) {
+          const int back = MAXT - 1 - j;
+          seen[j] = u[i + j][n];
+          if (rel < back)            // zeros in front of the taps, else the slot's row
+            seen[j] = back < taps && c < width && i < n_run
+                          ? *reinterpret_cast<const float2*>(tail + (long long)(rel - back + taps - 1) * C + c)
+                          : make_float2(0.f, 0.f);
+          y[n].x = fmaf(wt[n][j].x, seen[j].x, y[n].x);
+          y[n].y = fmaf(wt[n][j].y, seen[j].y, y[n].y);
+        }
+        if (move_tail && c < width && i < n_run) {     // the sequence's only token: what was read, one place on
+#pragma unroll
+          for (int j = 1; j < MAXT; j++) {
+            const int slot_row = j - (MAXT - taps) - 1;
+            if (slot_row >= 0) *reinterpret_cast<float2*>(tail + (long long)slot_row * C + c) = seen[j];
+          }
+        }
       }
-      continue;
     }
+#pragma unroll
+    for (int n = 0; n < NC; n++) u[i][n] = y[n];       // no later token reads this input
+  }
+  if (is_v) {
+#pragma unroll
+    for (int i = 0; i < R; i++) {
+      TO* dst = v_pool + __shfl_sync(0xffffffffu, my_dst, i);
+#pragma unroll
+      for (int n = 0; n < NC; n++) {
+        const int c = n * 64 + 2 * lane;
+        if (i < n_run && c < width) store2(dst + c, u[i][n].x, u[i][n].y);
+      }
+    }
+    return;
+  }
+#pragma unroll
+  for (int i = 0; i < R; i++) {
+    float ss = 0.f;
+#pragma unroll
+    for (int n = 0; n < NC; n++) ss = fmaf(u[i][n].x, u[i][n].x, fmaf(u[i][n].y, u[i][n].y, ss));
     const float inv = nw ? 1.0f / sqrtf(warp_sum(ss) / (float)p.hd + p.eps) : 1.0f;
 #pragma unroll
-    for (int n = 0; n < NC; n++) {
-      const int c = n * 64 + 2 * lane;
-      if (c < width) store2(buf + c, y[n].x * inv * norm_w[n].x, y[n].y * inv * norm_w[n].y);
-    }
-    __syncwarp();
-    TO* dst = is_q ? q_out + (long long)t * nq + col : k_pool + paged_offset(pk, seq, pos, head);
-    const float* tc = cs + (t - t0) * p.rot;
+    for (int n = 0; n < NC; n++)
+      store2(buf + i * (NC * 64) + n * 64 + 2 * lane, u[i][n].x * inv * norm_w[n].x, u[i][n].y * inv * norm_w[n].y);
+  }
+  __syncwarp();
+#pragma unroll
+  for (int i = 0; i < R; i++) {
+    TO* dst = (is_q ? q_out : k_pool) + __shfl_sync(0xffffffffu, my_dst, i);
+    const float* row = buf + i * (NC * 64);
+    const float* tc = cs + i * p.rot;
 #pragma unroll
     for (int n = 0; n < NC; n++) {
       const int c = n * 64 + 2 * lane;
-      if (c < width) {
+      if (i < n_run && c < width) {
         float o[2];
 #pragma unroll
         for (int e = 0; e < 2; e++) {
           const int ch = c + e;
-          const float own = buf[ch];
-          if (ch < half) o[e] = own * tc[ch] - buf[ch + half] * tc[half + ch];
-          else if (ch < p.rot) o[e] = own * tc[ch - half] + buf[ch - half] * tc[ch];
+          const float own = row[ch];
+          if (ch < half) o[e] = own * tc[ch] - row[ch + half] * tc[half + ch];
+          else if (ch < p.rot) o[e] = own * tc[ch - half] + row[ch - half] * tc[ch];
           else o[e] = own;
         }
         store2(dst + c, o[0], o[1]);
       }
     }
-    __syncwarp();              // the row is free for the next token
   }
-}
-
-template <typename TO, int TAPS>
-cudaError_t launch_taps(int nc, dim3 grid, size_t smem, cudaStream_t stream, const float* proj, int ld, const QkvConv& p,
-                        const float* w, float* state, long long state_stride, long long tail_off, const int* positions,
-                        const int* seq_of_token, const int* seq_q_start, const int* slots, const PagedView& pk,
-                        const PagedView& pvv, void* q_out, void* k_pool, void* v_pool, int T, int run, int move) {
-#define QC(NC)                                                                                                        \
-  return launch_dep(qkv_conv_kernel<TO, TAPS, NC>, grid, dim3(WARPS * 32), smem, stream, proj, ld, p, w, state,        \
-                    state_stride, tail_off, positions, seq_of_token, seq_q_start, slots, pk, pvv, (TO*)q_out,          \
-                    (TO*)k_pool, (TO*)v_pool, T, run, move)
-  if (nc <= 1) QC(1);
-  if (nc <= 2) QC(2);
-  QC(4);
-#undef QC
 }
 
 }  // namespace
@@ -191,6 +214,7 @@ MF_API int mf_qkv_conv_ok(int hd, int vd, int taps, int ld, int rot) {
          rot >= 0 && rot <= hd && rot % 2 == 0;
 }
 
+// w: [taps, channels] (a row per tap)
 MF_API int mf_qkv_conv(const float* proj, int ld, int out_dtype, int T, int n_heads, int n_kv, int hd, int vd, int rot,
                        float eps, const float* w, int taps, const float* q_w, const float* k_w, const float* inv_f,
                        const double* inv_d, float* state, long long state_stride, long long tail_off,
@@ -210,26 +234,29 @@ MF_API int mf_qkv_conv(const float* proj, int ld, int out_dtype, int T, int n_he
   const PagedView pvv{block_table, bt_stride, page_size, n_kv, vd};
   // one token from every sequence (the caller lays the step out so: T tokens of n_seqs sequences, none empty)
   const int single = (T == n_seqs && taps > 1) ? 1 : 0;
-  const int run = T >= 1024 ? 8 : T >= 128 ? 4 : 1;      // enough blocks first, then reuse
   const int widest = n_kv > 0 && vd > hd ? vd : hd;
-  const int nc = (widest + 63) / 64;
-  const size_t smem = (size_t)(run * rot + WARPS * (nc <= 1 ? 64 : nc <= 2 ? 128 : 256)) * sizeof(float);
+  const int nc = widest <= 64 ? 1 : widest <= 128 ? 2 : 4;
+  const int run = T < 128 ? 1 : nc == 4 ? 4 : 8;      // enough blocks first, then reuse
+  const size_t smem = (size_t)(run * rot + WARPS * run * nc * 64) * sizeof(float);
   const dim3 grid((T + run - 1) / run, (n_heads + 2 * n_kv + WARPS - 1) / WARPS);
   cudaError_t e;
-#define QT(TO, TAPS)                                                                                                  \
-  e = launch_taps<TO, TAPS>(nc, grid, smem, stream, proj, ld, p, w, state, state_stride, tail_off, positions,          \
-                            seq_of_token, seq_q_start, slots, pk, pvv, q_out, k_pool, v_pool, T, run, single)
+#define QC(TO, R, NC)                                                                                                 \
+  e = launch_dep(qkv_conv_kernel<TO, R, NC>, grid, dim3(WARPS * 32), smem, stream, proj, ld, p, w, taps, state,        \
+                 state_stride, tail_off, positions, seq_of_token, seq_q_start, slots, pk, pvv, (TO*)q_out,             \
+                 (TO*)k_pool, (TO*)v_pool, T, single)
 #define QA(TO)                                                                                                        \
   do {                                                                                                                \
-    if (taps == 1) QT(TO, 1);                                                                                         \
-    else if (taps == 2) QT(TO, 2);                                                                                    \
-    else if (taps == 3) QT(TO, 3);                                                                                    \
-    else QT(TO, 4);                                                                                                   \
+    if (nc == 1 && run == 1) QC(TO, 1, 1);                                                                            \
+    else if (nc == 1) QC(TO, 8, 1);                                                                                   \
+    else if (nc == 2 && run == 1) QC(TO, 1, 2);                                                                       \
+    else if (nc == 2) QC(TO, 8, 2);                                                                                   \
+    else if (run == 1) QC(TO, 1, 4);                                                                                  \
+    else QC(TO, 4, 4);                                                                                                \
   } while (0)
   if (out_dtype == MF_F32) QA(float);
   else QA(__nv_bfloat16);
 #undef QA
-#undef QT
+#undef QC
   if (e != cudaSuccess || taps == 1 || single) return (int)e;
   return (int)conv_tail_launch(proj, ld, C, taps, state, state_stride, tail_off, seq_q_start, seq_q_len, slots, n_seqs,
                                stream);

@@ -340,7 +340,7 @@ class NormedAttention(Mixer):
         if self.rotate_values:
             vf, vd = inverse_wavelengths(self.vd, base, runtime.device)
             self.vinv_f, self.vinv_d = vf, (vd if runtime.precise else None)
-        self.w_in = self.w_o = self.b_in = self.q_w = self.k_w = self.conv_w = self.sink = None
+        self.w_in = self.w_o = self.b_in = self.q_w = self.k_w = self.conv_w = self.conv_rows = self.sink = None
 
     def _n(self, role: str) -> str:
         return self.prefix + self.names[role]
@@ -393,6 +393,7 @@ class NormedAttention(Mixer):
             self.k_w = self.q_w if self.shares_cache else tensors[self._n("k_norm")].to(f32).contiguous()
         if self.taps:
             self.conv_w = torch.cat([tensors[self._n(r + "_conv")].to(f32) for r in self._roles()], dim=0).contiguous()
+            self.conv_rows = self.conv_w.t().contiguous()       # [taps, channels]: the fused kernel reads a row per tap
         if self.sink_value is not None:
             self.sink = torch.full((self.n_heads,), float(self.sink_value), dtype=f32, device=self.w_in.device)
 
@@ -413,7 +414,7 @@ class NormedAttention(Mixer):
             plain = (self.qk_norm != "whole" and not self.rotate_values and self.temp_coef == 0.0 and self.magnitude == 1.0
                      and (writes_cache or kv == 0))
             if plain and ops.qkv_conv_ok(self.hd, self.vd, self.taps, proj.shape[1], self.rot):
-                ops.qkv_conv(proj, self.n_heads, kv, self.hd, self.vd, self.rot, self.eps, self.conv_w, self.q_w,
+                ops.qkv_conv(proj, self.n_heads, kv, self.hd, self.vd, self.rot, self.eps, self.conv_rows, self.q_w,
                              self.k_w if kv else None, self.inv_f, self.inv_d, state, batch, table, cache.page_size, q,
                              cache.k, cache.v)
                 return
