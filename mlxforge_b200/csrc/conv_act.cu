@@ -124,17 +124,25 @@ conv_act_tail_kernel(const float* __restrict__ x, int ld, int C, int taps, float
   const int seq = blockIdx.x;
   const int start = seq_q_start[seq], n = seq_q_len[seq];
   float* tail = state + (long long)slots[seq] * state_stride + tail_off;
+  constexpr int AHEAD = 4;        // rows fetched before the first of them is written
   for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x)
-    for (int j = 0; j < taps - 1; j++) {          // ascending: a read is never behind a write
-      const int src = n - (taps - 1) + j;
-      tail[(long long)j * C + c] = src >= 0 ? x[(long long)(start + src) * ld + c] : tail[(long long)(j + n) * C + c];
+    for (int j0 = 0; j0 < taps - 1; j0 += AHEAD) {          // ascending: a read is never behind a write
+      float v[AHEAD];
+#pragma unroll
+      for (int e = 0; e < AHEAD; e++) {
+        const int j = j0 + e, src = n - (taps - 1) + j;
+        if (j < taps - 1) v[e] = src >= 0 ? x[(long long)(start + src) * ld + c] : tail[(long long)(j + n) * C + c];
+      }
+#pragma unroll
+      for (int e = 0; e < AHEAD; e++)
+        if (j0 + e < taps - 1) tail[(long long)(j0 + e) * C + c] = v[e];
     }
 }
 
 cudaError_t conv_tail_launch(const float* x, int ld, int C, int taps, float* state, long long state_stride,
                              long long tail_off, const int* seq_q_start, const int* seq_q_len, const int* slots, int n_seqs,
                              cudaStream_t stream) {
-  return launch_dep(conv_act_tail_kernel, dim3(n_seqs, (C + 1023) / 1024), dim3(256), 0, stream, x, ld, C, taps, state,
+  return launch_dep(conv_act_tail_kernel, dim3(n_seqs, (C + 255) / 256), dim3(256), 0, stream, x, ld, C, taps, state,
                     state_stride, tail_off, seq_q_start, seq_q_len, slots);
 }
 

@@ -8,8 +8,7 @@
 // deviations, or a root-mean-square norm, x / sqrt(mean(x^2) + eps); the two are chosen apart.  The
 // stream is 32-bit [T, H]; sums, deviations, norms and the add are 32-bit (the mean is taken first and
 // the squares are of the deviations) and out is rounded once.  With `rows` only those rows are
-// produced and the stream stays as it is.  One block per row; the order of the additions depends on H
-// alone.
+// produced and the stream stays as it is.  One block per row.
 #include "common.cuh"
 
 namespace {
@@ -82,9 +81,9 @@ post_norm_kernel(float* __restrict__ resid, const TY* __restrict__ y, const floa
 
 // ------------------------------------------------------------------ the serving case
 // bfloat16 output of the sublayer and of the norm in 16-byte pieces, H a multiple of 8 and at most
-// 8 * 256 * NV: every value stays in registers between the sums.
-template <int NV>
-__global__ void __launch_bounds__(256)
+// 8 * NT * NV: every value stays in registers between the sums.
+template <int NT, int NV>
+__global__ void __launch_bounds__(NT)
 post_norm_bf16_vec_kernel(float* __restrict__ resid, const __nv_bfloat16* __restrict__ y, const float* __restrict__ w1,
                           int kind1, float eps1, const float* __restrict__ w2, int kind2, float eps2,
                           __nv_bfloat16* __restrict__ out, const int* __restrict__ rows, int H) {
@@ -98,7 +97,7 @@ post_norm_bf16_vec_kernel(float* __restrict__ resid, const __nv_bfloat16* __rest
   float v[NV][8];
 #pragma unroll
   for (int j = 0; j < NV; j++) {
-    const int i = (j * 256 + threadIdx.x) * 8;
+    const int i = (j * NT + threadIdx.x) * 8;
 #pragma unroll
     for (int e = 0; e < 8; e++) v[j][e] = 0.f;
     if (i < H) {
@@ -113,7 +112,7 @@ post_norm_bf16_vec_kernel(float* __restrict__ resid, const __nv_bfloat16* __rest
     float s = 0.f;
 #pragma unroll
     for (int j = 0; j < NV; j++) {
-      const int i = (j * 256 + threadIdx.x) * 8;
+      const int i = (j * NT + threadIdx.x) * 8;
 #pragma unroll
       for (int e = 0; e < 8; e++) u[j][e] = 0.f;
       if (i < H) {
@@ -132,7 +131,7 @@ post_norm_bf16_vec_kernel(float* __restrict__ resid, const __nv_bfloat16* __rest
     float ss = 0.f;
 #pragma unroll
     for (int j = 0; j < NV; j++) {
-      if ((j * 256 + threadIdx.x) * 8 < H) {
+      if ((j * NT + threadIdx.x) * 8 < H) {
 #pragma unroll
         for (int e = 0; e < 8; e++) {
           u[j][e] -= mean;
@@ -143,7 +142,7 @@ post_norm_bf16_vec_kernel(float* __restrict__ resid, const __nv_bfloat16* __rest
     const float inv = kind1 == NK_NONE ? 1.0f : 1.0f / sqrtf(slot_sum(ss, red[1]) * inv_h + eps1);
 #pragma unroll
     for (int j = 0; j < NV; j++) {
-      const int i = (j * 256 + threadIdx.x) * 8;
+      const int i = (j * NT + threadIdx.x) * 8;
       if (i < H) {
 #pragma unroll
         for (int hf = 0; hf < 2; hf++) {
@@ -172,7 +171,7 @@ post_norm_bf16_vec_kernel(float* __restrict__ resid, const __nv_bfloat16* __rest
   float ss = 0.f;
 #pragma unroll
   for (int j = 0; j < NV; j++) {
-    if ((j * 256 + threadIdx.x) * 8 < H) {
+    if ((j * NT + threadIdx.x) * 8 < H) {
 #pragma unroll
       for (int e = 0; e < 8; e++) {
         v[j][e] -= mean;
@@ -184,7 +183,7 @@ post_norm_bf16_vec_kernel(float* __restrict__ resid, const __nv_bfloat16* __rest
   __nv_bfloat16* o = out + (long long)r * H;
 #pragma unroll
   for (int j = 0; j < NV; j++) {
-    const int i = (j * 256 + threadIdx.x) * 8;
+    const int i = (j * NT + threadIdx.x) * 8;
     if (i < H) {
       const float4 wa = *reinterpret_cast<const float4*>(w2 + i), wb = *reinterpret_cast<const float4*>(w2 + i + 4);
       uint4 pk;
@@ -211,12 +210,16 @@ MF_API int mf_post_norm(float* resid, const void* y, int y_dtype, const float* w
   mf_count(MF_K_POST_NORM);
   if (out_dtype == MF_BF16 && (!y || y_dtype == MF_BF16) && H % 8 == 0 && H <= 8 * 256 * 4 &&
       (((uintptr_t)resid | (uintptr_t)y | (uintptr_t)w1 | (uintptr_t)w2 | (uintptr_t)out) & 15) == 0) {
-#define PV(NV)                                                                                                       \
-  return (int)launch_dep(post_norm_bf16_vec_kernel<NV>, dim3(n_rows), dim3(256), 0, stream, resid,                    \
+#define PV(NT, NV)                                                                                                   \
+  return (int)launch_dep(post_norm_bf16_vec_kernel<NT, NV>, dim3(n_rows), dim3(NT), 0, stream, resid,                 \
                          (const __nv_bfloat16*)y, w1, kind1, eps1, w2, kind2, eps2, (__nv_bfloat16*)out, rows, H)
-    if (H <= 2048) PV(1);
-    if (H <= 4096) PV(2);
-    PV(4);
+    // many rows: few threads with many values each, as the four sums are what a row costs beside its bytes; few
+    // rows: many threads, as nothing else hides how long a thread takes
+    if (H <= 1024) PV(128, 1);
+    if (H <= 2048 && n_rows >= 256) PV(128, 2);
+    if (H <= 2048) PV(256, 1);
+    if (H <= 4096) PV(256, 2);
+    PV(256, 4);
 #undef PV
   }
   const size_t smem = (size_t)H * sizeof(float);

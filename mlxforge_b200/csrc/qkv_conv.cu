@@ -76,17 +76,17 @@ qkv_conv_kernel(const float* __restrict__ proj, int ld, QkvConv p, const float* 
   const int width = is_v ? p.vd : p.hd;
   const int col = is_q ? head * p.hd : is_v ? nq + nk + head * p.vd : nq + head * p.hd;
   const float* nw = is_v ? nullptr : is_q ? p.q_w : p.k_w;
-  float2 wt[NC][MAXT], norm_w[NC];
+  f32x2 wt[NC][MAXT], norm_w[NC];
 #pragma unroll
   for (int n = 0; n < NC; n++) {
     const int c = n * 64 + 2 * lane;
-    norm_w[n] = make_float2(1.f, 1.f);
+    norm_w[n] = pack2(1.f, 1.f);
     const bool in = live && c < width;
-    if (in && nw) norm_w[n] = make_float2(nw[c], nw[c + 1]);
+    if (in && nw) norm_w[n] = pack2(nw[c], nw[c + 1]);
 #pragma unroll
     for (int j = 0; j < MAXT; j++) {
       const int tap = j - (MAXT - taps);
-      wt[n][j] = in && tap >= 0 ? *reinterpret_cast<const float2*>(w + (long long)tap * C + col + c) : make_float2(0.f, 0.f);
+      wt[n][j] = in && tap >= 0 ? *reinterpret_cast<const f32x2*>(w + (long long)tap * C + col + c) : 0ull;
     }
   }
   // lane i looks up token i of the run: its distance from the first token its sequence brings, its slot and
@@ -103,7 +103,7 @@ qkv_conv_kernel(const float* __restrict__ proj, int ld, QkvConv p, const float* 
   pdl_wait();
   if (!live) return;
   // u[i + MAXT - 1] is token i of the run; what stands before it is used by the tokens of its own sequence only
-  float2 u[R + MAXT - 1][NC];
+  f32x2 u[R + MAXT - 1][NC];
 #pragma unroll
   for (int i = 0; i < R + MAXT - 1; i++) {
     const int t = t0 + i - (MAXT - 1);
@@ -111,22 +111,21 @@ qkv_conv_kernel(const float* __restrict__ proj, int ld, QkvConv p, const float* 
 #pragma unroll
     for (int n = 0; n < NC; n++) {
       const int c = n * 64 + 2 * lane;
-      u[i][n] = row && c < width ? *reinterpret_cast<const float2*>(proj + (long long)t * ld + col + c) : make_float2(0.f, 0.f);
+      u[i][n] = row && c < width ? *reinterpret_cast<const f32x2*>(proj + (long long)t * ld + col + c) : 0ull;
     }
   }
 #pragma unroll
   for (int i = 0; i < R; i++) {
     const int rel = __shfl_sync(0xffffffffu, my_rel, i);
-    float2 y[NC];
+    f32x2 y[NC];
     if (rel >= taps - 1) {           // every input is among the rows of this step
 #pragma unroll
       for (int n = 0; n < NC; n++) {
-        y[n] = make_float2(0.f, 0.f);
+        y[n] = 0ull;
 #pragma unroll
         for (int j = 0; j < MAXT; j++) {
           if (j < MAXT - taps) continue;          // a padded tap: another sequence's row may stand there
-          y[n].x = fmaf(wt[n][j].x, u[i + j][n].x, y[n].x);
-          y[n].y = fmaf(wt[n][j].y, u[i + j][n].y, y[n].y);
+          y[n] = fma2(wt[n][j], u[i + j][n], y[n]);
         }
       }
     } else {                         // the first tokens of a portion: the slot has what came before
@@ -134,24 +133,23 @@ qkv_conv_kernel(const float* __restrict__ proj, int ld, QkvConv p, const float* 
 #pragma unroll
       for (int n = 0; n < NC; n++) {
         const int c = n * 64 + 2 * lane;
-        y[n] = make_float2(0.f, 0.f);
-        float2 seen[MAXT];
+        y[n] = 0ull;
+        f32x2 seen[MAXT];
 #pragma unroll
         for (int j = 0; j < MAXT; j++) {
           const int back = MAXT - 1 - j;
           seen[j] = u[i + j][n];
           if (rel < back)            // zeros in front of the taps, else the slot's row
             seen[j] = back < taps && c < width && i < n_run
-                          ? *reinterpret_cast<const float2*>(tail + (long long)(rel - back + taps - 1) * C + c)
-                          : make_float2(0.f, 0.f);
-          y[n].x = fmaf(wt[n][j].x, seen[j].x, y[n].x);
-          y[n].y = fmaf(wt[n][j].y, seen[j].y, y[n].y);
+                          ? *reinterpret_cast<const f32x2*>(tail + (long long)(rel - back + taps - 1) * C + c)
+                          : 0ull;
+          if (j >= MAXT - taps) y[n] = fma2(wt[n][j], seen[j], y[n]);
         }
         if (move_tail && c < width && i < n_run) {     // the sequence's only token: what was read, one place on
 #pragma unroll
           for (int j = 1; j < MAXT; j++) {
             const int slot_row = j - (MAXT - taps) - 1;
-            if (slot_row >= 0) *reinterpret_cast<float2*>(tail + (long long)slot_row * C + c) = seen[j];
+            if (slot_row >= 0) *reinterpret_cast<f32x2*>(tail + (long long)slot_row * C + c) = seen[j];
           }
         }
       }
@@ -166,22 +164,38 @@ qkv_conv_kernel(const float* __restrict__ proj, int ld, QkvConv p, const float* 
 #pragma unroll
       for (int n = 0; n < NC; n++) {
         const int c = n * 64 + 2 * lane;
-        if (i < n_run && c < width) store2(dst + c, u[i][n].x, u[i][n].y);
+        const float2 v = unpack2(u[i][n]);
+        if (i < n_run && c < width) store2(dst + c, v.x, v.y);
       }
     }
     return;
   }
+  // lane i gets token i's sum of squares, so that the root and the division are done once
+  float mine = 1.0f;
+  if (nw) {
+#pragma unroll
+    for (int i = 0; i < R; i++) {
+      f32x2 sq = 0ull;
+#pragma unroll
+      for (int n = 0; n < NC; n++) sq = fma2(u[i][n], u[i][n], sq);
+      const float2 h = unpack2(sq);
+      const float total = warp_sum(h.x + h.y);
+      if (lane == i) mine = total;
+    }
+    mine = 1.0f / sqrtf(mine / (float)p.hd + p.eps);
+  }
 #pragma unroll
   for (int i = 0; i < R; i++) {
-    float ss = 0.f;
+    const float inv = __shfl_sync(0xffffffffu, mine, i);
+    const f32x2 inv2 = pack2(inv, inv);
 #pragma unroll
-    for (int n = 0; n < NC; n++) ss = fmaf(u[i][n].x, u[i][n].x, fmaf(u[i][n].y, u[i][n].y, ss));
-    const float inv = nw ? 1.0f / sqrtf(warp_sum(ss) / (float)p.hd + p.eps) : 1.0f;
-#pragma unroll
-    for (int n = 0; n < NC; n++)
-      store2(buf + i * (NC * 64) + n * 64 + 2 * lane, u[i][n].x * inv * norm_w[n].x, u[i][n].y * inv * norm_w[n].y);
+    for (int n = 0; n < NC; n++) {
+      u[i][n] = mul2(mul2(u[i][n], inv2), norm_w[n]);
+      if (n * 64 < p.rot) *reinterpret_cast<f32x2*>(buf + i * (NC * 64) + n * 64 + 2 * lane) = u[i][n];
+    }
   }
   __syncwarp();
+  const bool even = (half & 1) == 0;           // both channels of a lane then stand on one side of a pair
 #pragma unroll
   for (int i = 0; i < R; i++) {
     TO* dst = (is_q ? q_out : k_pool) + __shfl_sync(0xffffffffu, my_dst, i);
@@ -190,17 +204,29 @@ qkv_conv_kernel(const float* __restrict__ proj, int ld, QkvConv p, const float* 
 #pragma unroll
     for (int n = 0; n < NC; n++) {
       const int c = n * 64 + 2 * lane;
-      if (i < n_run && c < width) {
-        float o[2];
+      if (i >= n_run || c >= width) continue;
+      f32x2 o = u[i][n];
+      if (even) {
+        if (c < p.rot) {
+          const bool first = c < half;
+          const int j = first ? c : c - half;
+          f32x2 sn = *reinterpret_cast<const f32x2*>(tc + half + j);
+          if (first) sn = mul2(sn, pack2(-1.f, -1.f));
+          o = fma2(o, *reinterpret_cast<const f32x2*>(tc + j),
+                   mul2(*reinterpret_cast<const f32x2*>(row + (first ? c + half : j)), sn));
+        }
+        const float2 v = unpack2(o);
+        store2(dst + c, v.x, v.y);
+      } else {
+        const float2 own = unpack2(o);
+        float v[2] = {own.x, own.y};
 #pragma unroll
         for (int e = 0; e < 2; e++) {
           const int ch = c + e;
-          const float own = row[ch];
-          if (ch < half) o[e] = own * tc[ch] - row[ch + half] * tc[half + ch];
-          else if (ch < p.rot) o[e] = own * tc[ch - half] + row[ch - half] * tc[ch];
-          else o[e] = own;
+          if (ch < half) v[e] = v[e] * tc[ch] - row[ch + half] * tc[half + ch];
+          else if (ch < p.rot) v[e] = v[e] * tc[ch - half] + row[ch - half] * tc[ch];
         }
-        store2(dst + c, o[0], o[1]);
+        store2(dst + c, v[0], v[1]);
       }
     }
   }
